@@ -8,6 +8,8 @@ wherever its mixer is defined (a test file is enough): the manager has no list o
 A *paged* kind stores something for every token, in pages that the manager hands out; its answers:
   window(need)                          -> tokens that stay readable (None: all); needs with equal windows share a
                                            group, i.e. a pool of page ids and one block table per request
+  chunk(need)       (optional)          -> instead of a window: the size of the runs of positions, counted from a request's
+                                           start, outside of which nothing is read (None)
   keep_first(need)  (optional)          -> tokens at the start of a request that stay readable behind the window (0);
                                            needs of one group agree on it too
   page_shape(need, page_size)           -> shape of one page of one cache slot
@@ -48,6 +50,9 @@ class PagedKVKind:
     def window(self, need):
         return need.window
 
+    def chunk(self, need):
+        return getattr(need, "chunk", None)
+
     def keep_first(self, need):
         return int(getattr(need, "keep_first", 0) or 0) if need.window is not None else 0
 
@@ -81,19 +86,36 @@ class FixedStateKind:
 
 
 def lifetime_of(need, kind):
-    """What names a paged need's group: its window alone, or (window, kept first tokens) when some are kept.  The
-    window and the kept tokens themselves are `lifetime_window` and `lifetime_keep` of that key."""
+    """What names a paged need's group: its window alone, (window, kept first tokens) when some are kept, or
+    ("chunk", size).  The reach in tokens, the kept tokens and whether it is chunks are `lifetime_window`,
+    `lifetime_keep` and `lifetime_chunked` of that key."""
+    chunk = kind.chunk(need) if hasattr(kind, "chunk") else None
+    if chunk is not None:
+        return ("chunk", int(chunk))
     window = kind.window(need)
     keep = int(kind.keep_first(need)) if (window is not None and hasattr(kind, "keep_first")) else 0
     return (window, keep) if keep > 0 else window
 
 
+def lifetime_chunked(key) -> bool:
+    return isinstance(key, tuple) and key[0] == "chunk"
+
+
 def lifetime_window(key):
+    if lifetime_chunked(key):
+        return key[1]
     return key[0] if isinstance(key, tuple) else key
 
 
 def lifetime_keep(key) -> int:
-    return key[1] if isinstance(key, tuple) else 0
+    return key[1] if isinstance(key, tuple) and not lifetime_chunked(key) else 0
+
+
+def lifetime_name(key) -> str:
+    """The key in words, without spaces: none, 96, 96+4 (four kept tokens), chunk200."""
+    if lifetime_chunked(key):
+        return f"chunk{key[1]}"
+    return "none" if key is None else (f"{key[0]}+{key[1]}" if isinstance(key, tuple) else str(key))
 
 
 def flatten_need(need) -> list:

@@ -13,7 +13,7 @@ declaration-driven shape but stores tokens in fixed-size pages:
 * pages return to the pool when the request is released, and in a windowed group as soon as every
   position they hold is out of reach of any later query: a query at position p reads keys
   j >= p - window + 1, so after a step that leaves the request at length n the pages that end at or
-  before n - window + 1 go back;
+  before n - window + 1 go back (in a group of chunks of C positions: at or before floor(n / C) * C);
 * every live request also owns one state slot (an index into dense per-request state arrays) for
   mixers that keep a state of fixed size; it is zeroed at admission.
 
@@ -28,7 +28,7 @@ import numpy as np
 import torch
 
 from ..parts.base import StateBundle
-from .kinds import FixedStateView, PagedKVView, flatten_need, kind_of, lifetime_keep, lifetime_of, lifetime_window       # the views are re-exported from here
+from .kinds import FixedStateView, PagedKVView, flatten_need, kind_of, lifetime_chunked, lifetime_keep, lifetime_of, lifetime_window       # the views are re-exported from here
 
 _OK, _E_NOT_LIVE, _E_ALREADY_LIVE, _E_NO_SLOT, _E_OUT_OF_PAGES, _E_CONTEXT, _E_COMMIT, _E_PAGE, _E_INCONSISTENT = range(9)
 
@@ -57,10 +57,10 @@ def host_library():
         lib.kf_cache_pool_n_taken.argtypes = [ctypes.c_void_p, ctypes.c_int]
         for name in ("kf_pool_destroy", "kf_pool_take", "kf_pool_give_back", "kf_pool_n_free", "kf_pool_is_held",
                      "kf_cache_destroy", "kf_cache_width", "kf_cache_n_live", "kf_cache_pool_n_free",
-                     "kf_cache_pool_is_held", "kf_cache_mirror", "kf_cache_check"):
+                     "kf_cache_pool_is_held", "kf_cache_mirror", "kf_cache_check", "kf_cache_chunked"):
             getattr(lib, name).argtypes = [ctypes.c_void_p] + [ctypes.c_int] * {"kf_pool_give_back": 1, "kf_pool_is_held": 1,
                                                                                   "kf_cache_pool_n_free": 1, "kf_cache_pool_is_held": 2,
-                                                                                  "kf_cache_mirror": 1}.get(name, 0)
+                                                                                  "kf_cache_mirror": 1, "kf_cache_chunked": 1}.get(name, 0)
         i64 = ctypes.c_int64
         for name, extra in (("kf_cache_contains", []), ("kf_cache_length", []), ("kf_cache_state_slot", []),
                             ("kf_cache_add_request", []), ("kf_cache_cancel_reservation", []), ("kf_cache_release", []),
@@ -216,6 +216,8 @@ class CacheManager:
         self._h = ctypes.c_void_p(self._lib.kf_cache_create(G, windows, sizes, self.page_size, self.max_requests,
                                                             self.max_context))
         for gi, g in enumerate(self.groups):
+            if lifetime_chunked(g.window):
+                self._lib.kf_cache_chunked(self._h, gi)
             if lifetime_keep(g.window) > 0:
                 self._lib.kf_cache_keep_first(self._h, gi, int(lifetime_keep(g.window)))
         self.table_width = self._lib.kf_cache_width(self._h)

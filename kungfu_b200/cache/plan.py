@@ -8,6 +8,7 @@ device cannot hold it (crates/kf-engine/src/plan.rs:199-228,319-343).  With page
 * a request can hold at most `ctx` tokens in a group without a window, and at most `window + batch + page` tokens in
   a windowed group (the keys the earliest row of its next portion still reads, the portion itself, and one page of
   slack because pages are given back whole); a pool never needs more than `parallel` times that;
+* a group of chunks of C positions is sized like a window of C;
 * the pools of all groups together must fit the memory budget; if they do not, every group is cut by the same
   factor, but never below what ONE request of full context needs (below that nothing can run: `NoFit`).
 
@@ -55,11 +56,12 @@ class CachePlan:
 
     def fields(self) -> dict:
         """Flat key/values for the `plan` event line."""
+        from .kinds import lifetime_name
         out = {"page_size": self.page_size, "parallel": self.parallel, "ctx": self.ctx, "batch": self.batch,
                "cache_bytes": self.total_bytes, "budget_bytes": self.budget_bytes if self.budget_bytes is not None else "none",
                "shrunk": int(self.shrunk)}
         for i, g in enumerate(self.groups):
-            out[f"group{i}"] = f"window:{g.window if g.window is not None else 'none'},pages:{g.pages},tokens_per_request:{g.tokens_per_request},slots:{len(g.slots)}"
+            out[f"group{i}"] = f"window:{lifetime_name(g.window)},pages:{g.pages},tokens_per_request:{g.tokens_per_request},slots:{len(g.slots)}"
         return out
 
 
@@ -81,7 +83,7 @@ def plan_cache(needs: list, *, page_size: int, parallel: int, ctx: int, batch: i
         if not kind.paged:
             fixed += parallel * kind.fixed_bytes(need)
             continue
-        window = lifetime_of(need, kind)             # the group's key: the window, or (window, kept first tokens)
+        window = lifetime_of(need, kind)             # the group's key: the window, (window, kept first tokens) or ("chunk", size)
         g = groups.get(window)
         if g is None:
             if window is None:

@@ -191,7 +191,7 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
     return;
   }
   const int pos = positions[t];
-  const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+  const int lo = kf_first_key(pos, window);
   const int n_keys = pos + 1 - lo;
   int per = (n_keys + n_splits - 1) / n_splits;
   per = (per + 63) & ~63;                                     // whole 64-key runs per split
@@ -360,14 +360,17 @@ constexpr int DM_KEYS = 16;                       // keys per warp tile
 // position rotates the new key, writes key and value into the page (if `write_kv`) and then reads them like any other.
 // What does not depend on earlier kernels of the step (the step's integers, keys of earlier steps) is requested
 // before the grid dependency is waited for.
-template <int D>
+//
+// SIG: no softmax.  Key j counts with sigmoid(s_j + sig_bias[h]) and the weights are not normalized: the weighted sum is
+// what is stored.  In the merges this is a maximum of 0 everywhere and a sum of 1 that the first split holds.
+template <int D, bool SIG>
 __global__ void __launch_bounds__(DM_WARPS * 32)
 attn_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, const float* __restrict__ qkv, const float* __restrict__ cos_t,
                        const float* __restrict__ sin_t, int rot, int write_kv, __nv_bfloat16* pages,
                        const int* __restrict__ items, int n_items, const int* __restrict__ positions,
                        const int* __restrict__ row_req, const int* __restrict__ table, int table_stride, int page_size,
                        int nh, int nkv, float scale, float softcap, int window, int vsplit, int keep_first, int sink,
-                       int n_splits, float* __restrict__ partial, int* __restrict__ counters,
+                       const float* __restrict__ sig_bias, int n_splits, float* __restrict__ partial, int* __restrict__ counters,
                        __nv_bfloat16* __restrict__ out) {
   using namespace kf_mma;
   kf_pdl_trigger();
@@ -400,7 +403,7 @@ attn_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, const float* __restr
     return;
   }
   const int pos = positions[t];
-  const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+  const int lo = kf_first_key(pos, window);
   // Kept first tokens: keys [0, kept) are seen behind the window.  The keys are walked by a running index u in
   // [lo_v, pos]: u >= lo is key u itself, u in [lo_v, lo) is key u - lo_v, so the walk below does not know of the gap.
   const int kept = window > 0 ? min(keep_first, lo) : 0;
@@ -522,6 +525,12 @@ attn_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, const float* __restr
   for (int n = 0; n < NT_O; ++n) { o_acc[n][0] = o_acc[n][1] = o_acc[n][2] = o_acc[n][3] = 0.f; }
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
   const float cap2 = softcap > 0.f ? 2.f * LOG2E / softcap : 0.f;
+  float sb[2] = {0.f, 0.f};                                        // the bias of this thread's two heads, in base-2 units
+  if (SIG) {
+#pragma unroll
+    for (int r = 0; r < 2; ++r)
+      if (g + r * 8 < G) sb[r] = sig_bias[h_first + g + r * 8] * LOG2E;
+  }
 
   int buf = 0;                                                     // buffer of the item in use: item n is in n % DM_BUFS
   for (int it = 0; it < n_mine; ++it) {
@@ -573,36 +582,42 @@ attn_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, const float* __restr
           const float ex = exp2f(s * cap2);
           s = softcap * (1.f - __fdividef(2.f, ex + 1.f));
         }
-        s = (j < k_end) ? s * LOG2E : -INFINITY;
-        s_acc[n][e] = s;
-        m_new[r] = fmaxf(m_new[r], s);
+        if (SIG) {
+          s_acc[n][e] = (j < k_end) ? __fdividef(1.f, 1.f + exp2f(-fmaxf(fmaf(s, LOG2E, sb[r]), -120.f))) : 0.f;
+        } else {
+          s = (j < k_end) ? s * LOG2E : -INFINITY;
+          s_acc[n][e] = s;
+          m_new[r] = fmaxf(m_new[r], s);
+        }
       }
     }
-    float corr[2];
+    if constexpr (!SIG) {
+      float corr[2];
 #pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      m_new[r] = fmaxf(m_new[r], __shfl_xor_sync(0xffffffffu, m_new[r], 1));
-      m_new[r] = fmaxf(m_new[r], __shfl_xor_sync(0xffffffffu, m_new[r], 2));
-      corr[r] = (m_new[r] == -INFINITY) ? 1.f : exp2f(m_run[r] - m_new[r]);
-      m_run[r] = m_new[r];
-    }
-    float l_add[2] = {0.f, 0.f};
-#pragma unroll
-    for (int n = 0; n < 2; ++n) {
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int r = e >> 1;
-        const float p = (m_new[r] == -INFINITY) ? 0.f : exp2f(s_acc[n][e] - m_new[r]);
-        s_acc[n][e] = p;
-        l_add[r] += p;
+      for (int r = 0; r < 2; ++r) {
+        m_new[r] = fmaxf(m_new[r], __shfl_xor_sync(0xffffffffu, m_new[r], 1));
+        m_new[r] = fmaxf(m_new[r], __shfl_xor_sync(0xffffffffu, m_new[r], 2));
+        corr[r] = (m_new[r] == -INFINITY) ? 1.f : exp2f(m_run[r] - m_new[r]);
+        m_run[r] = m_new[r];
       }
-    }
+      float l_add[2] = {0.f, 0.f};
 #pragma unroll
-    for (int r = 0; r < 2; ++r) l_run[r] = l_run[r] * corr[r] + l_add[r];
+      for (int n = 0; n < 2; ++n) {
 #pragma unroll
-    for (int n = 0; n < NT_O; ++n) {
-      o_acc[n][0] *= corr[0]; o_acc[n][1] *= corr[0];
-      o_acc[n][2] *= corr[1]; o_acc[n][3] *= corr[1];
+        for (int e = 0; e < 4; ++e) {
+          const int r = e >> 1;
+          const float p = (m_new[r] == -INFINITY) ? 0.f : exp2f(s_acc[n][e] - m_new[r]);
+          s_acc[n][e] = p;
+          l_add[r] += p;
+        }
+      }
+#pragma unroll
+      for (int r = 0; r < 2; ++r) l_run[r] = l_run[r] * corr[r] + l_add[r];
+#pragma unroll
+      for (int n = 0; n < NT_O; ++n) {
+        o_acc[n][0] *= corr[0]; o_acc[n][1] *= corr[0];
+        o_acc[n][2] *= corr[1]; o_acc[n][3] *= corr[1];
+      }
     }
     uint32_t a[4];
     a[0] = pack_bf16(s_acc[0][0], s_acc[0][1]);
@@ -644,7 +659,7 @@ attn_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, const float* __restr
         dst[0] = o_acc[n][2 * r];
         dst[1] = o_acc[n][2 * r + 1];
       }
-      if (tq == 0) { sm_ml[warp][row][0] = m_run[r]; sm_ml[warp][row][1] = l_run[r]; }
+      if (tq == 0) { sm_ml[warp][row][0] = SIG ? 0.f : m_run[r]; sm_ml[warp][row][1] = SIG ? (warp == 0 && split == 0) : l_run[r]; }
     }
   }
   __syncthreads();
@@ -684,14 +699,14 @@ attn_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, const float* __restr
 
 // Blocks of the tensor-core decode kernel that one SM holds at a time (shared memory or registers, whichever binds), as
 // the runtime reports it; also sets the kernel's shared-memory limit.  0 if that fails.
-template <int D>
+template <int D, bool SIG>
 int decode_mma_blocks_per_sm() {
   static int cached = -1;
   if (cached >= 0) return cached;
   const size_t smem = (size_t)(16 * D + DM_WARPS * DM_BUFS * DM_KEYS * D) * 2;
   int n = 0;
-  if (cudaFuncSetAttribute(attn_decode_mma_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess ||
-      cudaOccupancyMaxActiveBlocksPerMultiprocessor(&n, attn_decode_mma_kernel<D>, DM_WARPS * 32, smem) != cudaSuccess) {
+  if (cudaFuncSetAttribute(attn_decode_mma_kernel<D, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess ||
+      cudaOccupancyMaxActiveBlocksPerMultiprocessor(&n, attn_decode_mma_kernel<D, SIG>, DM_WARPS * 32, smem) != cudaSuccess) {
     kf_record_cuda_error(cudaGetLastError());
     return 0;
   }
@@ -699,17 +714,17 @@ int decode_mma_blocks_per_sm() {
   return n;
 }
 
-template <int D>
+template <int D, bool SIG>
 int launch_decode_mma(const float* qkv, const float* cos_t, const float* sin_t, int rot, int write_kv,
                       const void* q, const void* pages, const int* items, int n_items, const int* positions,
                       const int* row_req, const int* table, int table_stride, int page_size, int nh, int nkv, float scale,
-                      float softcap, int window, int vsplit, int keep_first, int sink, int n_splits, float* partial, int* counters,
-                      void* out, cudaStream_t stream) {
+                      float softcap, int window, int vsplit, int keep_first, int sink, const float* sig_bias, int n_splits,
+                      float* partial, int* counters, void* out, cudaStream_t stream) {
   const size_t smem = (size_t)(16 * D + DM_WARPS * DM_BUFS * DM_KEYS * D) * 2;
-  if (decode_mma_blocks_per_sm<D>() < 1) return KF_ERR_SETUP;
-  kf_launch(attn_decode_mma_kernel<D>, dim3(n_items * nkv, n_splits), dim3(DM_WARPS * 32), smem, stream,
+  if (decode_mma_blocks_per_sm<D, SIG>() < 1) return KF_ERR_SETUP;
+  kf_launch(attn_decode_mma_kernel<D, SIG>, dim3(n_items * nkv, n_splits), dim3(DM_WARPS * 32), smem, stream,
             (const __nv_bfloat16*)q, qkv, cos_t, sin_t, rot, write_kv, (__nv_bfloat16*)const_cast<void*>(pages), items, n_items,
-            positions, row_req, table, table_stride, page_size, nh, nkv, scale, softcap, window, vsplit, keep_first, sink, n_splits,
+            positions, row_req, table, table_stride, page_size, nh, nkv, scale, softcap, window, vsplit, keep_first, sink, sig_bias, n_splits,
             partial, counters, (__nv_bfloat16*)out);
   KF_CHECK_LAUNCH();
   return KF_OK;
@@ -752,9 +767,9 @@ KF_API int kf_attention_decode_mma_plan(int n_items, int nh, int nkv, int d, int
   if (g_forced_splits > 0) { *splits_out = g_forced_splits; return KF_OK; }
   const long blocks = (long)n_items * nkv;
   // fill one wave: as many splits as resident blocks allow
-  long per_sm = d == 256 ? decode_mma_blocks_per_sm<256>() : d == 128 ? decode_mma_blocks_per_sm<128>()
-              : d == 64 ? decode_mma_blocks_per_sm<64>() : d == 32 ? decode_mma_blocks_per_sm<32>()
-              : d == 16 ? decode_mma_blocks_per_sm<16>() : 0;
+  long per_sm = d == 256 ? decode_mma_blocks_per_sm<256, false>() : d == 128 ? decode_mma_blocks_per_sm<128, false>()
+              : d == 64 ? decode_mma_blocks_per_sm<64, false>() : d == 32 ? decode_mma_blocks_per_sm<32, false>()
+              : d == 16 ? decode_mma_blocks_per_sm<16, false>() : 0;
   if (per_sm > 8) per_sm = 8;
   if (per_sm < 1) per_sm = 1;
   int splits = (int)((kf_sm_count() * per_sm) / blocks);
@@ -790,22 +805,24 @@ KF_API int kf_attention_decode(const void* q, void* out, const void* pages, cons
                                const int* positions, const int* row_req, const int* table, int table_stride,
                                int page_size, int nh, int nkv, int d, float scale, float softcap, int window, int vsplit,
                                int ht, int n_splits, float* partial, int* counters, int keep_first, int sink,
-                               cudaStream_t stream) {
+                               const float* sig_bias, cudaStream_t stream) {
   if (n_items <= 0) return KF_OK;
-  if ((keep_first > 0 || sink) && ht != 0) return KF_ERR_SIZE;     // kept first tokens and the sink: tensor-core variant only
+  if ((keep_first > 0 || sink || sig_bias) && ht != 0) return KF_ERR_SIZE;   // kept first tokens, the sink, sigmoid weights: tensor-core variant only
   if (window <= 0) keep_first = 0;
   if (nkv < 1 || nh % nkv != 0 || page_size < 1 || n_splits < 1 || !kf_head_map_ok(nh, nkv, vsplit)) return KF_ERR_SIZE;
   if (n_splits > 1 && (!partial || !counters)) return KF_ERR_SIZE;
   if (n_splits > MERGE_MAX_SPLITS || ht > MERGE_MAX_HEADS) return KF_ERR_SIZE;
   if (ht == 0) {                                     // tensor-core variant
     if (nh / nkv > 16) return KF_ERR_SIZE;
-#define KF_MMA_ARGS nullptr, nullptr, nullptr, 0, 0, q, pages, items, n_items, positions, row_req, table, table_stride, page_size, nh, nkv, scale, softcap, window, vsplit, keep_first, sink, n_splits, partial, counters, out, stream
+#define KF_MMA_ARGS nullptr, nullptr, nullptr, 0, 0, q, pages, items, n_items, positions, row_req, table, table_stride, page_size, nh, nkv, scale, softcap, window, vsplit, keep_first, sink, sig_bias, n_splits, partial, counters, out, stream
     switch (d) {
-      case 16: return launch_decode_mma<16>(KF_MMA_ARGS);
-      case 32: return launch_decode_mma<32>(KF_MMA_ARGS);
-      case 64: return launch_decode_mma<64>(KF_MMA_ARGS);
-      case 128: return launch_decode_mma<128>(KF_MMA_ARGS);
-      case 256: return launch_decode_mma<256>(KF_MMA_ARGS);
+#define KF_MMA(DD) (sig_bias ? launch_decode_mma<DD, true>(KF_MMA_ARGS) : launch_decode_mma<DD, false>(KF_MMA_ARGS))
+      case 16: return KF_MMA(16);
+      case 32: return KF_MMA(32);
+      case 64: return KF_MMA(64);
+      case 128: return KF_MMA(128);
+      case 256: return KF_MMA(256);
+#undef KF_MMA
     }
 #undef KF_MMA_ARGS
     return KF_ERR_SIZE;
@@ -835,13 +852,13 @@ KF_API int kf_attention_decode_fused(const float* qkv, const float* cos_t, const
   if (rot < 0 || rot > d || (rot & 1) || (rot > 0 && (!cos_t || !sin_t))) return KF_ERR_SIZE;
   if (n_splits > 1 && (!partial || !counters)) return KF_ERR_SIZE;
   if (n_splits > MERGE_MAX_SPLITS) return KF_ERR_SIZE;
-#define KF_MMA_ARGS qkv, cos_t, sin_t, rot, write_kv, nullptr, pages, items, n_items, positions, row_req, table, table_stride, page_size, nh, nkv, scale, softcap, window, 0, 0, 0, n_splits, partial, counters, out, stream
+#define KF_MMA_ARGS qkv, cos_t, sin_t, rot, write_kv, nullptr, pages, items, n_items, positions, row_req, table, table_stride, page_size, nh, nkv, scale, softcap, window, 0, 0, 0, nullptr, n_splits, partial, counters, out, stream
   switch (d) {
-    case 16: return launch_decode_mma<16>(KF_MMA_ARGS);
-    case 32: return launch_decode_mma<32>(KF_MMA_ARGS);
-    case 64: return launch_decode_mma<64>(KF_MMA_ARGS);
-    case 128: return launch_decode_mma<128>(KF_MMA_ARGS);
-    case 256: return launch_decode_mma<256>(KF_MMA_ARGS);
+    case 16: return launch_decode_mma<16, false>(KF_MMA_ARGS);
+    case 32: return launch_decode_mma<32, false>(KF_MMA_ARGS);
+    case 64: return launch_decode_mma<64, false>(KF_MMA_ARGS);
+    case 128: return launch_decode_mma<128, false>(KF_MMA_ARGS);
+    case 256: return launch_decode_mma<256, false>(KF_MMA_ARGS);
   }
 #undef KF_MMA_ARGS
   return KF_ERR_SIZE;
@@ -918,5 +935,5 @@ KF_API int kf_attention_decode_static(const void* q, void* out, const void* page
     }
   }
   return kf_attention_decode(q, out, pages, nullptr, n_rows, positions, row_req, table, table_stride, page_size, nh, nkv,
-                             d, scale, softcap, window, 0, ht, splits, partial, counters, 0, 0, stream);
+                             d, scale, softcap, window, 0, ht, splits, partial, counters, 0, 0, nullptr, stream);
 }

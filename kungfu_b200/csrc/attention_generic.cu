@@ -9,6 +9,8 @@
 // keep_first > 0 (with a window): keys 0..keep_first-1 stay visible behind the window, at their true positions, so the
 // warp walks [0, min(keep_first, lo)) and then [lo, p].  sink != 0: the softmax's denominator has one more term, exp(0)
 // (a key of score 0 without a value): the walk starts from maximum 0 and sum 1.
+// window < 0: chunks of -window positions (kf_first_key).  sig_bias (one number per head, or null): no softmax; key j counts
+// with sigmoid(s_j + sig_bias[h]), and the weights are not normalized.
 // The order of every sum is fixed by (row, head) alone, so a row's result does not depend on how the
 // step was cut or what else is in the batch.  This is the engine's 32-bit attention and the fallback of
 // the bfloat16 path for head sizes the tensor-core kernels do not take.
@@ -23,7 +25,7 @@ attention_generic_kernel(const TQ* __restrict__ q, TQ* __restrict__ out, const T
                          const int* __restrict__ items, const int* __restrict__ positions,
                          const int* __restrict__ row_req, const int* __restrict__ block_table, int table_stride,
                          int page_size, int nh, int nkv, int d, float scale, float softcap, int window, int vsplit,
-                         int keep_first, int sink, int T) {
+                         int keep_first, int sink, const float* __restrict__ sig_bias, int T) {
   kf_pdl_trigger();
   kf_pdl_wait();
   __shared__ float qs[WARPS][MAX_D];
@@ -41,7 +43,7 @@ attention_generic_kernel(const TQ* __restrict__ q, TQ* __restrict__ out, const T
   const int kvh = h / (nh / nkv);
   const KfHeadMap hm = kf_head_map(h, kvh, nh, nkv, vsplit);
   const int pos = positions[t];
-  const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+  const int lo = kf_first_key(pos, window);
   const TQ* qr = q + ((size_t)t * hm.n_query + hm.query) * d;
   for (int i = lane; i < d; i += 32) qs[warp][i] = kf_load(qr, i);
   __syncwarp();
@@ -69,12 +71,18 @@ attention_generic_kernel(const TQ* __restrict__ q, TQ* __restrict__ out, const T
         for (int i = 0; i < d; ++i) dot = fmaf(qs[warp][i], kf_load(kr, i), dot);
         s = kf_softcap(dot * scale, softcap);
       }
-      const float m_new = fmaxf(m, kf_warp_max(s));
-      const float p = valid ? expf(s - m_new) : 0.f;
-      const float corr = (m == -INFINITY) ? 0.f : expf(m - m_new);
-      l = l * corr + kf_warp_sum(p);
+      float m_new, p;
+      if (sig_bias) {
+        m_new = 0.f, l = 1.f;
+        p = valid ? 1.f / (1.f + expf(-(s + sig_bias[h]))) : 0.f;
+      } else {
+        m_new = fmaxf(m, kf_warp_max(s));
+        p = valid ? expf(s - m_new) : 0.f;
+        const float corr = (m == -INFINITY) ? 0.f : expf(m - m_new);
+        l = l * corr + kf_warp_sum(p);
 #pragma unroll
-      for (int r = 0; r < MAX_D / 32; ++r) acc[r] *= corr;
+        for (int r = 0; r < MAX_D / 32; ++r) acc[r] *= corr;
+      }
       const int n = min(32, last - c0 + 1);
       for (int u = 0; u < n; ++u) {
         const float pu = __shfl_sync(0xffffffffu, p, u);
@@ -101,7 +109,7 @@ attention_generic_kernel(const TQ* __restrict__ q, TQ* __restrict__ out, const T
 KF_API int kf_attention_generic(const void* q, void* out, int q_dtype, const void* pages, int kv_dtype,
                                 const int* items, const int* positions, const int* row_req, const int* block_table, int table_stride,
                                 int page_size, int nh, int nkv, int d, float scale, float softcap, int window,
-                                int vsplit, int keep_first, int sink, int T, cudaStream_t stream) {
+                                int vsplit, int keep_first, int sink, const float* sig_bias, int T, cudaStream_t stream) {
   if (T <= 0) return KF_OK;
   if (d < 1 || d > MAX_D_ALL || nkv < 1 || nh % nkv != 0 || page_size < 1 || !kf_head_map_ok(nh, nkv, vsplit)) return KF_ERR_SIZE;
   const long n_work = (long)T * nh;
@@ -109,7 +117,7 @@ KF_API int kf_attention_generic(const void* q, void* out, int q_dtype, const voi
 #define KF_GO1(TQ, TKV, MAXD)                                                                              \
   kf_launch(attention_generic_kernel<TQ, TKV, MAXD>, dim3(blocks), dim3(WARPS * 32), 0, stream,                               \
       (const TQ*)q, (TQ*)out, (const TKV*)pages, items, positions, row_req, block_table, table_stride, page_size, \
-      nh, nkv, d, scale, softcap, window, vsplit, window > 0 ? keep_first : 0, sink, T)
+      nh, nkv, d, scale, softcap, window, vsplit, window > 0 ? keep_first : 0, sink, sig_bias, T)
 #define KF_GO(TQ, TKV) do { if (d <= 256) KF_GO1(TQ, TKV, 256); else KF_GO1(TQ, TKV, 512); } while (0)
   if (q_dtype == KF_F32 && kv_dtype == KF_F32) KF_GO(float, float);
   else if (q_dtype == KF_BF16 && kv_dtype == KF_BF16) KF_GO(__nv_bfloat16, __nv_bfloat16);

@@ -21,14 +21,15 @@ using namespace kf_mma;
 constexpr int BM = 64;                 // query rows per tile
 constexpr int PF_WARPS = 4;
 
-template <int D, int BNK>
+// SIG: no softmax; key j counts with sigmoid(s_j + sig_bias[h]) and the weights are not normalized.
+template <int D, int BNK, bool SIG>
 __global__ void __launch_bounds__(PF_WARPS * 32)
 attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ pages,
                     const int* __restrict__ tile_row0, const int* __restrict__ tile_nrows,
                     const int* __restrict__ positions, const int* __restrict__ row_req,
                     const int* __restrict__ table, int table_stride, int page_size, int nh, int nkv,
                     float scale, float softcap, int window, int vsplit, int keep_first, int sink,
-                    __nv_bfloat16* __restrict__ out) {
+                    const float* __restrict__ sig_bias, __nv_bfloat16* __restrict__ out) {
   kf_pdl_trigger();
   kf_pdl_wait();
   constexpr int CH = D / 8;                       // 16-byte chunks per row
@@ -49,7 +50,7 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
   const KfHeadMap hm = kf_head_map(h, kvh, nh, nkv, vsplit);
   const int pos0 = positions[row0];                               // rows of a request are consecutive positions
   const int pos_last = pos0 + nrows - 1;
-  const int lo = (window > 0 && pos0 - window + 1 > 0) ? pos0 - window + 1 : 0;
+  const int lo = kf_first_key(pos0, window);
   const int kt_begin = (lo / BNK) * BNK;
   // kept first tokens that lie before the first tile of the window: their tiles are walked first (the mask below lets a
   // row see key j < keep_first wherever its window stands)
@@ -95,6 +96,8 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
   float m_run[2] = {sink ? 0.f : -INFINITY, sink ? 0.f : -INFINITY};
   float l_run[2] = {(sink && (lane & 3) == 0) ? 1.f : 0.f, (sink && (lane & 3) == 0) ? 1.f : 0.f};
   const int prow[2] = {pos0 + warp * 16 + g, pos0 + warp * 16 + g + 8};   // positions of this thread's two rows
+  const int first_key_of[2] = {kf_first_key(prow[0], window), kf_first_key(prow[1], window)};
+  const float sb = SIG ? sig_bias[h] * LOG2E : 0.f;
   const float cap2 = softcap > 0.f ? 2.f * LOG2E / softcap : 0.f;
 
   for (int it = 0; it < n_ktiles; ++it) {
@@ -137,12 +140,17 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
           const float ex = exp2f(s * cap2);
           s = softcap * (1.f - __fdividef(2.f, ex + 1.f));
         }
-        const bool seen = j <= prow[r] && (window <= 0 || prow[r] - j < window || j < keep_first);
+        const bool seen = j <= prow[r] && (j >= first_key_of[r] || j < keep_first);
+        if (SIG) {
+          s_acc[n][e] = seen ? __fdividef(1.f, 1.f + exp2f(-fmaxf(fmaf(s, LOG2E, sb), -120.f))) : 0.f;
+          continue;
+        }
         s = seen ? s * LOG2E : -INFINITY;
         s_acc[n][e] = s;
         m_new[r] = fmaxf(m_new[r], s);
       }
     }
+    if constexpr (!SIG) {
     float corr[2];
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
@@ -168,6 +176,7 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
     for (int n = 0; n < NT_O; ++n) {
       o_acc[n][0] *= corr[0]; o_acc[n][1] *= corr[0];
       o_acc[n][2] *= corr[1]; o_acc[n][3] *= corr[1];
+    }
     }
     // ---- O += P V -----------------------------------------------------------------------------------------------
 #pragma unroll
@@ -199,7 +208,7 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
   for (int r = 0; r < 2; ++r) {
     const int lr = warp * 16 + g + r * 8;
     if (lr >= nrows) continue;
-    const float inv = l_run[r] > 0.f ? 1.f / l_run[r] : 0.f;
+    const float inv = SIG ? 1.f : (l_run[r] > 0.f ? 1.f / l_run[r] : 0.f);
     __nv_bfloat16* orow = out + ((size_t)(row0 + lr) * nh + h) * D;
 #pragma unroll
     for (int n = 0; n < NT_O; ++n) {
@@ -209,23 +218,23 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
   }
 }
 
-template <int D, int BNK>
+template <int D, int BNK, bool SIG>
 int launch_prefill(const void* q, void* out, const void* pages, const int* tile_row0, const int* tile_nrows, int n_tiles,
                    const int* positions, const int* row_req, const int* table, int table_stride, int page_size,
                    int nh, int nkv, float scale, float softcap, int window, int vsplit, int keep_first, int sink,
-                   cudaStream_t stream) {
+                   const float* sig_bias, cudaStream_t stream) {
   const size_t smem = (size_t)(BM * D + 4 * BNK * D) * 2;
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(attn_prefill_kernel<D, BNK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+    if (cudaFuncSetAttribute(attn_prefill_kernel<D, BNK, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
       kf_record_cuda_error(cudaGetLastError());
       return KF_ERR_SETUP;
     }
     configured = true;
   }
-  kf_launch(attn_prefill_kernel<D, BNK>, dim3(n_tiles, nh), dim3(PF_WARPS * 32), smem, stream, 
+  kf_launch(attn_prefill_kernel<D, BNK, SIG>, dim3(n_tiles, nh), dim3(PF_WARPS * 32), smem, stream, 
       (const __nv_bfloat16*)q, (const __nv_bfloat16*)pages, tile_row0, tile_nrows, positions, row_req, table, table_stride,
-      page_size, nh, nkv, scale, softcap, window, vsplit, window > 0 ? keep_first : 0, sink, (__nv_bfloat16*)out);
+      page_size, nh, nkv, scale, softcap, window, vsplit, window > 0 ? keep_first : 0, sink, sig_bias, (__nv_bfloat16*)out);
   KF_CHECK_LAUNCH();
   return KF_OK;
 }
@@ -240,17 +249,19 @@ KF_API int kf_attention_prefill_tile_rows() { return BM; }
 KF_API int kf_attention_prefill(const void* q, void* out, const void* pages, const int* tile_row0, const int* tile_nrows,
                                 int n_tiles, const int* positions, const int* row_req, const int* table, int table_stride,
                                 int page_size, int nh, int nkv, int d, float scale, float softcap, int window, int vsplit,
-                                int keep_first, int sink, cudaStream_t stream) {
+                                int keep_first, int sink, const float* sig_bias, cudaStream_t stream) {
   if (n_tiles <= 0) return KF_OK;
   if (nkv < 1 || nh % nkv != 0 || page_size < 1 || !kf_head_map_ok(nh, nkv, vsplit)) return KF_ERR_SIZE;
-#define KF_ARGS q, out, pages, tile_row0, tile_nrows, n_tiles, positions, row_req, table, table_stride, page_size, nh, nkv, scale, softcap, window, vsplit, keep_first, sink, stream
+#define KF_ARGS q, out, pages, tile_row0, tile_nrows, n_tiles, positions, row_req, table, table_stride, page_size, nh, nkv, scale, softcap, window, vsplit, keep_first, sink, sig_bias, stream
+#define KF_PF(DD, BB) (sig_bias ? launch_prefill<DD, BB, true>(KF_ARGS) : launch_prefill<DD, BB, false>(KF_ARGS))
   switch (d) {
-    case 16: return launch_prefill<16, 64>(KF_ARGS);
-    case 32: return launch_prefill<32, 64>(KF_ARGS);
-    case 64: return launch_prefill<64, 64>(KF_ARGS);
-    case 128: return launch_prefill<128, 64>(KF_ARGS);
-    case 256: return launch_prefill<256, 32>(KF_ARGS);
+    case 16: return KF_PF(16, 64);
+    case 32: return KF_PF(32, 64);
+    case 64: return KF_PF(64, 64);
+    case 128: return KF_PF(128, 64);
+    case 256: return KF_PF(256, 32);
   }
+#undef KF_PF
 #undef KF_ARGS
   return KF_ERR_SIZE;
 }

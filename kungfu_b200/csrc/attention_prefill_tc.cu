@@ -192,7 +192,7 @@ __device__ __forceinline__ void tmem_st16(uint32_t taddr, const float* v) {
 __device__ __forceinline__ int tile_key_tiles(int row0, int nrows, const int* positions, const int* row_req, int window,
                                               int keep_first, int* kt_first, int* n_kept) {
   const int pos0 = positions[row0];
-  const int lo = (window > 0 && pos0 - window + 1 > 0) ? pos0 - window + 1 : 0;
+  const int lo = kf_first_key(pos0, window);
   *kt_first = (lo / BKV) * BKV;
   *n_kept = (window > 0 && keep_first > 0) ? (min(keep_first, *kt_first) + BKV - 1) / BKV : 0;
   return (row_req[row0] < 0 || nrows <= 0) ? 0 : *n_kept + (pos0 + nrows - 1 - *kt_first) / BKV + 1;   // padding, or a tile without rows
@@ -207,14 +207,16 @@ __device__ __forceinline__ int tile_runs(int n_key_tiles, int n_parts, int run_t
   return p < 1 ? 1 : (p > n_parts ? n_parts : p);
 }
 
-template <int D>
+// SIG: no softmax.  Key j counts with sigmoid(s_j + sig_bias[h]) and the weights are not normalized, so there is no running
+// maximum to hand over and O is never rescaled; for the merge of runs a row's maximum is 0 and the first run holds a sum of 1.
+template <int D, bool SIG>
 __global__ void __launch_bounds__(THREADS, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_kv,
                        const int* __restrict__ tile_row0, const int* __restrict__ tile_nrows,
                        const int* __restrict__ positions, const int* __restrict__ row_req,
                        const int* __restrict__ table, int table_stride, int page_size, int nh, int nkv,
                        float scale, float softcap, int window, int vsplit, int keep_first, int sink,
-                       __nv_bfloat16* __restrict__ out, int* __restrict__ error_flag, int n_parts, int run_tiles,
+                       const float* __restrict__ sig_bias, __nv_bfloat16* __restrict__ out, int* __restrict__ error_flag, int n_parts, int run_tiles,
                        float* __restrict__ partial) {
   constexpr int NSUB = D / 64;                            // 64-element sub-tiles along the head dimension
   constexpr int Q_BYTES = BMQ * D * 2;
@@ -387,6 +389,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
     const float c3 = softcap * LOG2E;
     const float ct = softcap > 0.f ? scale / softcap : 0.f;
     const float c4 = c3 * ct;
+    const int row_lo = kf_first_key(prow, window);         // this row's first visible key
+    const int warp_lo = kf_first_key(pos0 + wq * 32 + 31, window);   // a key from here on is seen by every row of the warp below it
+    const float sb = SIG ? sig_bias[h] * LOG2E : 0.f;
     constexpr int HC = D / 2;                              // O columns of this thread in the epilogue
     float m_mine = -INFINITY, l_sum = 0.f;                 // this group's sum of exponentials, scaled to 2^-m_mine
     bool ok = true;
@@ -402,7 +407,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
       mbar_arrive(&s_free[grp]);                           // the buffer may take the scores of tile i + 2
       // Scores in base-2 units: s2 = log2(e) * cap * tanh(scale * s / cap) = c3 - 2 c3 / (exp2(s * c1) + 1), or
       // s * c0 without a cap.  A tile that every row of this warp sees whole skips the mask.
-      const bool whole = (kt + BKV - 1 <= pos0 + wq * 32) && (window <= 0 || pos0 + wq * 32 + 31 - kt < window);
+      const bool whole = (kt + BKV - 1 <= pos0 + wq * 32) && kt >= warp_lo;
       if (softcap > 0.f) {
         // A cap is chosen beyond what scores usually reach: while every score of this warp's tile is within it
         // (|scale * s / cap| <= 1), tanh is a polynomial on the packed 32-bit pipe; otherwise it goes through exp2 and
@@ -431,7 +436,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
       if (!whole) {
         // key kt + c is seen by this row iff first <= c <= last: one bit per key, tested with constant masks
         const int last = prow - kt;                                        // >= 64: all of the tile
-        const int first = window > 0 ? last - window + 1 : 0;              // <= 0: from the tile's first key
+        const int first = row_lo - kt;                                     // <= 0: from the tile's first key
         const unsigned long long causal = last < 0 ? 0ull : (last >= 63 ? ~0ull : ((2ull << last) - 1ull));
         unsigned long long seen = causal;
         if (first > 0) seen &= first >= 64 ? 0ull : ~((1ull << first) - 1ull);
@@ -446,6 +451,30 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
           sv[32 + c] = (seen_hi & (1u << c)) ? sv[32 + c] : -INFINITY;
         }
       }
+      uint32_t pk[BKV / 2];
+      bool raise = false;
+      float corr = 1.f;
+      if constexpr (SIG) {
+        // 1 / (1 + 2^-x) for four keys at a time with ONE reciprocal: of the product of the four denominators, which the
+        // clamp keeps below 2^122 (a weight is then at least 2^-30); masked keys (x = -inf) are zeroed afterwards
+#pragma unroll
+        for (int c = 0; c < BKV; c += 4) {
+          float dn[4];
+#pragma unroll
+          for (int e = 0; e < 4; ++e) dn[e] = 1.f + ex2_fast(fminf(-(sv[c + e] + sb), 30.f));
+          const float d01 = dn[0] * dn[1], d23 = dn[2] * dn[3];
+          const float rr = rcp_fast(d01 * d23);
+          const float r01 = rr * d23, r23 = rr * d01;
+          float w[4] = {r01 * dn[1], r01 * dn[0], r23 * dn[3], r23 * dn[2]};
+          if (!whole) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) w[e] = sv[c + e] == -INFINITY ? 0.f : w[e];
+          }
+          const __nv_bfloat162 b0 = __floats2bfloat162_rn(w[0], w[1]), b1 = __floats2bfloat162_rn(w[2], w[3]);
+          pk[c >> 1] = *reinterpret_cast<const uint32_t*>(&b0);
+          pk[(c >> 1) + 1] = *reinterpret_cast<const uint32_t*>(&b1);
+        }
+      } else {
       float mt[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
       for (int c = 0; c < BKV; c += 8) {
@@ -456,16 +485,15 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
       // the maximum O is scaled to after tile i - 1, from the other group; this tile's goes back the same way
       if (i > 0) ok = ok && mbar_wait(&m_done[grp ^ 1], ((i - 1) >> 1) & 1);
       const float m_used = i > 0 ? s_max[r] : -INFINITY;
-      const bool raise = m_tile > m_used + RESCALE_STEP;   // also true for the first finite maximum
+      raise = m_tile > m_used + RESCALE_STEP;   // also true for the first finite maximum
       const float m_new = raise ? m_tile : m_used;
       s_max[r] = m_new;
       mbar_arrive(&m_done[grp]);
-      const float corr = raise ? ex2_fast(m_used - m_new) : 1.f;   // for O; exp2(-inf) = 0 when nothing was accumulated yet
+      corr = raise ? ex2_fast(m_used - m_new) : 1.f;   // for O; exp2(-inf) = 0 when nothing was accumulated yet
       const float m_sub = (m_new == -INFINITY) ? 0.f : m_new;      // a row that has seen nothing yet: exp2(-inf - 0) = 0
       const float l_corr = (m_mine == m_new) ? 1.f : ex2_fast(m_mine - m_new);   // this group's sum follows the maximum
       float2 la[4] = {{0.f, 0.f}, {0.f, 0.f}, {0.f, 0.f}, {0.f, 0.f}};   // four chains of packed sums; the order is fixed
       const float2 neg_m = make_float2(-m_sub, -m_sub);
-      uint32_t pk[BKV / 2];
 #pragma unroll
       for (int c = 0; c < BKV; c += 2) {
         const float2 x = __fadd2_rn(make_float2(sv[c], sv[c + 1]), neg_m);
@@ -476,10 +504,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
       }
       l_sum = l_sum * l_corr + (((la[0].x + la[0].y) + (la[1].x + la[1].y)) + ((la[2].x + la[2].y) + (la[3].x + la[3].y)));
       m_mine = m_new;
+      }
       if (i > 0) {                                          // P V of the previous tile must be done: O is at rest, P is free
         ok = ok && mbar_wait(&pv_done[(i - 1) & 1], ((i - 1) >> 1) & 1);
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-        if (__any_sync(0xffffffffu, raise)) {              // rescale this row of O (all lanes of the warp take part)
+        if (!SIG && __any_sync(0xffffffffu, raise)) {              // rescale this row of O (all lanes of the warp take part)
 #pragma unroll 1
           for (int c = 0; c < D; c += 16) {
             float o[16];
@@ -505,14 +534,19 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
     if (ok && n_tiles > 0) ok = mbar_wait(&pv_done[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1);
     if (!ok) { atomicExch(error_flag, ERR_ATTN_WAIT + 3); *s_abort = 1; }
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+    float m_used = 0.f;
+    if constexpr (!SIG) {
     // the row's sum is the two groups' sums, both brought to the last maximum; every softmax thread reaches this
     asm volatile("bar.sync 2, 256;" ::: "memory");          // every tile's maximum has been published
-    const float m_used = n_tiles > 0 ? s_max[r] : -INFINITY;
+    m_used = n_tiles > 0 ? s_max[r] : -INFINITY;
     l_sum = (m_mine == m_used) ? l_sum : l_sum * ex2_fast(m_mine - m_used);
     asm volatile("bar.sync 2, 256;" ::: "memory");          // ... and read by both threads of the row
     s_max[half * BMQ + r] = l_sum;
     asm volatile("bar.sync 2, 256;" ::: "memory");
     l_sum = s_max[r] + s_max[BMQ + r];
+    } else {
+      l_sum = part == 0 ? 1.f : 0.f;
+    }
     // the sink (a key of score 0 without a value) adds 2^(0 - m) to the sum of the run that holds the walk's first tile
     // (a run whose scores all lie far below zero, or that this row sees nothing of, leaves the sink alone: maximum 0, sum 1)
     float m_rec = m_used;
@@ -526,7 +560,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
     } else if (my_parts > 1) {
       // ---- one of several runs of keys: leave O as it is (scaled by 2^-m), with m and the sum, for the merge ----------
       const bool run_ok = __all_sync(0xffffffffu, ok && n_tiles > 0 && *s_abort == 0);
-      const bool have = run_ok && r < nrows && l_sum > 0.f;     // a row that saw no key in this run leaves m = -inf
+      const bool have = run_ok && r < nrows && (SIG || l_sum > 0.f);     // a row that saw no key in this run leaves m = -inf
       float* rec = partial + (((size_t)(row0 + (r < nrows ? r : 0)) * nh + h) * n_parts + part) * (D + 4);
       if (half == 0 && r < nrows) { rec[D] = have ? m_rec : -INFINITY; rec[D + 1] = have ? l_sum : 0.f; }
       if (run_ok) {
@@ -659,22 +693,22 @@ bool tensor_map(const void* base, long rows, long cols, int box_rows, CUtensorMa
   return true;
 }
 
-template <int D>
+template <int D, bool SIG>
 int launch(const CUtensorMap& tq, const CUtensorMap& tkv, const int* tile_row0, const int* tile_nrows, int n_tiles,
            const int* positions, const int* row_req, const int* table, int table_stride, int page_size, int nh, int nkv,
-           float scale, float softcap, int window, int vsplit, int keep_first, int sink, void* out, int* error_flag,
+           float scale, float softcap, int window, int vsplit, int keep_first, int sink, const float* sig_bias, void* out, int* error_flag,
            int n_parts, int run_tiles, float* partial, cudaStream_t stream) {
   const size_t smem = (size_t)BMQ * D * 2 + 4 * (size_t)BKV * D * 2 + (size_t)BMQ * BKV * 2 + 1024 + 256 + 4 * BMQ * 4;
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(attn_prefill_tc_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+    if (cudaFuncSetAttribute(attn_prefill_tc_kernel<D, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
       kf_record_cuda_error(cudaGetLastError());
       return KF_ERR_SETUP;
     }
     configured = true;
   }
-  kf_launch(attn_prefill_tc_kernel<D>, dim3(n_tiles * n_parts * nh), dim3(THREADS), smem, stream, tq, tkv, tile_row0, tile_nrows,
-            positions, row_req, table, table_stride, page_size, nh, nkv, scale, softcap, window, vsplit, keep_first, sink,
+  kf_launch(attn_prefill_tc_kernel<D, SIG>, dim3(n_tiles * n_parts * nh), dim3(THREADS), smem, stream, tq, tkv, tile_row0, tile_nrows,
+            positions, row_req, table, table_stride, page_size, nh, nkv, scale, softcap, window, vsplit, keep_first, sink, sig_bias,
             (__nv_bfloat16*)out, error_flag, n_parts, run_tiles, partial);
   KF_CHECK_LAUNCH();
   if (n_parts > 1) {
@@ -737,7 +771,7 @@ KF_API int kf_attention_prefill_tc(const void* q, void* out, const void* pages, 
                                    const int* tile_nrows, int n_tiles, const int* positions, const int* row_req,
                                    const int* table, int table_stride, int page_size, int nh, int nkv, int d, float scale,
                                    float softcap, int window, int vsplit, int* error_flag, int n_parts, int run_tiles,
-                                   float* partial, int keep_first, int sink, cudaStream_t stream) {
+                                   float* partial, int keep_first, int sink, const float* sig_bias, cudaStream_t stream) {
   if (n_tiles <= 0) return KF_OK;
   if (window <= 0) keep_first = 0;
   if (nkv < 1 || nh % nkv != 0 || page_size % 64 != 0 || !kf_head_map_ok(nh, nkv, vsplit)) return KF_ERR_SIZE;
@@ -746,12 +780,14 @@ KF_API int kf_attention_prefill_tc(const void* q, void* out, const void* pages, 
   CUtensorMap tq, tkv;
   if (!tensor_map(q, T, (long)hm.n_query * d, BMQ, &tq)) return KF_ERR_SETUP;
   if (!tensor_map(pages, n_pages * 2 * hm.n_stored * page_size, d, BKV, &tkv)) return KF_ERR_SETUP;
-#define KF_ARGS tq, tkv, tile_row0, tile_nrows, n_tiles, positions, row_req, table, table_stride, page_size, nh, nkv, scale, softcap, window, vsplit, keep_first, sink, out, error_flag, n_parts, run_tiles, partial, stream
+#define KF_ARGS tq, tkv, tile_row0, tile_nrows, n_tiles, positions, row_req, table, table_stride, page_size, nh, nkv, scale, softcap, window, vsplit, keep_first, sink, sig_bias, out, error_flag, n_parts, run_tiles, partial, stream
+#define KF_TC(DD) (sig_bias ? launch<DD, true>(KF_ARGS) : launch<DD, false>(KF_ARGS))
   switch (d) {
-    case 64: return launch<64>(KF_ARGS);
-    case 128: return launch<128>(KF_ARGS);
-    case 256: return launch<256>(KF_ARGS);
+    case 64: return KF_TC(64);
+    case 128: return KF_TC(128);
+    case 256: return KF_TC(256);
   }
+#undef KF_TC
 #undef KF_ARGS
   return KF_ERR_SIZE;
 }

@@ -121,6 +121,16 @@ __device__ __forceinline__ float kf_clamped_swish(float g, float u, float limit)
 
 __device__ __forceinline__ float kf_softcap(float x, float cap) { return cap > 0.f ? cap * tanhf(x / cap) : x; }
 
+// Which keys the row at position p sees besides j <= p, as one integer in every attention kernel's arguments:
+//   mask > 0   a sliding window: p - j < mask
+//   mask < 0   chunks of -mask positions, counted from 0: p and j stand in the same chunk
+//   mask = 0   every key
+// All three are a first visible key that never falls as p rises.
+__host__ __device__ __forceinline__ int kf_first_key(int p, int mask) {
+  if (mask > 0) return p - mask + 1 > 0 ? p - mask + 1 : 0;
+  return mask < 0 ? p - p % (-mask) : 0;
+}
+
 static inline int kf_ceil_div(long a, long b) { return (int)((a + b - 1) / b); }
 
 // Which stored heads an attention head reads.  Ordinarily (vsplit = 0) the nh heads of a row of q and of the result are

@@ -297,12 +297,67 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, const TW* __r
   }
 }
 
+// The same for long heads (a norm over all heads of a row at once is one head): a block per (row, head), the head in
+// registers, NPT elements per thread.
+template <typename TW, typename TO, int NPT>
+__global__ void __launch_bounds__(512)
+head_norm_gate_block_kernel(const float* o, const TW* __restrict__ w, float eps, const float* gate, int ld_gate, int gate0,
+                            int act, TO* __restrict__ out, int H, int dv, int w_stride, int ldo, int ocol0, float scale) {
+  kf_pdl_trigger();
+  __shared__ float red[33];
+  const int t = blockIdx.x / H, h = blockIdx.x - t * H;
+  float wv[NPT], v[NPT], z[NPT];
+#pragma unroll
+  for (int k = 0; k < NPT; ++k) {
+    const int i = threadIdx.x + k * blockDim.x;
+    wv[k] = i < dv ? kf_load(w, h * w_stride + i) : 0.f;
+  }
+  kf_pdl_wait();
+  o = kf_produced(o), gate = kf_produced(gate);
+  const float* src = o + ((size_t)t * H + h) * dv;
+  const float* g = gate + (size_t)t * ld_gate + gate0 + h * dv;
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < NPT; ++k) {
+    const int i = threadIdx.x + k * blockDim.x;
+    v[k] = i < dv ? src[i] : 0.f;
+    z[k] = i < dv ? g[i] : 0.f;
+    ss = fmaf(v[k], v[k], ss);
+  }
+  ss = kf_block_sum(ss, red);
+  const float inv = 1.f / sqrtf(ss / (float)dv + eps);
+  TO* dst = out + (size_t)t * ldo + ocol0 + h * dv;
+#pragma unroll
+  for (int k = 0; k < NPT; ++k) {
+    const int i = threadIdx.x + k * blockDim.x;
+    if (i >= dv) continue;
+    const float s = 1.f / (1.f + expf(-z[k]));
+    kf_store(dst, i, v[k] * inv * wv[k] * (act == 0 ? z[k] * s : s) * scale);
+  }
+}
+
 KF_API int kf_head_norm_gate(const float* o, const void* w, int w_dtype, float eps, const float* gate, int ld_gate, int gate0,
                              int act, void* out, int out_dtype, int H, int dv, int T, int w_stride, int ldo, int ocol0, float scale,
                              cudaStream_t stream) {
   if (T <= 0) return KF_OK;
   if (ldo <= 0) ldo = H * dv;                   // rows of `out` hold the heads alone
   if (ocol0 < 0 || ocol0 + H * dv > ldo) return KF_ERR_SIZE;
+  if (dv >= 512 && dv <= 8192) {
+    const int threads = dv >= 2048 ? 512 : 256, npt = kf_ceil_div(dv, threads);
+#define KF_BLOCK(TW, TO, NPT)                                                                                             \
+  kf_launch(head_norm_gate_block_kernel<TW, TO, NPT>, dim3((unsigned)((long)T * H)), dim3(threads), 0, stream, o, (const TW*)w, eps, \
+            gate, ld_gate, gate0, act, (TO*)out, H, dv, w_stride, ldo, ocol0, scale)
+#define KF_GO(TW, TO) do { if (npt <= 4) KF_BLOCK(TW, TO, 4); else if (npt <= 8) KF_BLOCK(TW, TO, 8); else KF_BLOCK(TW, TO, 16); } while (0)
+    if (w_dtype == KF_F32 && out_dtype == KF_F32) KF_GO(float, float);
+    else if (w_dtype == KF_BF16 && out_dtype == KF_BF16) KF_GO(__nv_bfloat16, __nv_bfloat16);
+    else if (w_dtype == KF_BF16 && out_dtype == KF_F32) KF_GO(__nv_bfloat16, float);
+    else if (w_dtype == KF_F32 && out_dtype == KF_BF16) KF_GO(float, __nv_bfloat16);
+    else return KF_ERR_DTYPE;
+#undef KF_GO
+#undef KF_BLOCK
+    KF_CHECK_LAUNCH();
+    return KF_OK;
+  }
   const dim3 grid(kf_ceil_div((long)T * H, 4));
 #define KF_GO(TW, TO) \
   kf_launch(head_norm_gate_kernel<TW, TO>, grid, dim3(128), 0, stream, o, (const TW*)w, eps, gate, ld_gate, gate0, act, (TO*)out, H, dv, T, w_stride, ldo, ocol0, scale)

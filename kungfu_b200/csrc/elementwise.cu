@@ -31,6 +31,62 @@ KF_API int kf_embed(const int* tokens, const void* table, int table_dtype, float
   return KF_OK;
 }
 
+// x[t, :] = table[token[t], :] * scale + pair[row(t), :], a second table read by the token and the one before it:
+// row(t) = (previous * mul_prev + token * mul_cur) mod buckets in 64-bit integers, the table's last row (number `buckets`)
+// for a request's first token.  The previous token of a step's first row of a request is its state, prev[slot] (written
+// here too: the block of that row is the only one that reads or writes it).  Padding rows (request -1) give zeros.
+template <typename TW>
+__global__ void embed_pair_kernel(const int* __restrict__ tokens, const TW* __restrict__ table, const TW* __restrict__ pair,
+                                  float scale, long long mul_prev, long long mul_cur, long long buckets, int* prev,
+                                  float* __restrict__ out, int H, int V, const int* __restrict__ positions,
+                                  const int* __restrict__ row_req, const int* __restrict__ req_row_start,
+                                  const int* __restrict__ req_n_rows, const int* __restrict__ req_state_slot, int writes) {
+  kf_pdl_trigger();
+  kf_pdl_wait();
+  __shared__ long long s_row;
+  const int t = blockIdx.x, req = row_req[t];
+  float* o = out + (size_t)t * H;
+  if (req < 0) {
+    for (int i = threadIdx.x; i < H; i += blockDim.x) o[i] = 0.f;
+    return;
+  }
+  const int tok = tokens[t];
+  if (threadIdx.x == 0) {
+    const int row0 = req_row_start[req], slot = req_state_slot[req];
+    long long r = buckets;
+    if (positions[t] > 0) {
+      const long long before = t > row0 ? tokens[t - 1] : prev[slot];
+      r = (before * mul_prev + (long long)tok * mul_cur) % buckets;
+      if (r < 0) r += buckets;
+    }
+    s_row = r;
+    if (t == row0 && writes) prev[slot] = tokens[row0 + req_n_rows[req] - 1];
+  }
+  __syncthreads();
+  const bool ok = tok >= 0 && tok < V;
+  const TW* a = table + (size_t)(ok ? tok : 0) * H;
+  const TW* b = pair + (size_t)s_row * H;
+  for (int i = threadIdx.x; i < H; i += blockDim.x) o[i] = ok ? kf_load(a, i) * scale + kf_load(b, i) : 0.f;
+}
+
+KF_API int kf_embed_pair(const int* tokens, const void* table, const void* pair, int dtype, float scale, long long mul_prev,
+                         long long mul_cur, long long buckets, int* prev, float* out, int T, int H, int V, const int* positions,
+                         const int* row_req, const int* req_row_start, const int* req_n_rows, const int* req_state_slot,
+                         int writes, cudaStream_t stream) {
+  if (T <= 0) return KF_OK;
+  if (buckets < 1 || !prev) return KF_ERR_SIZE;
+  const int threads = H >= 1024 ? 256 : 128;
+#define KF_GO(TW)                                                                                                          \
+  kf_launch(embed_pair_kernel<TW>, dim3(T), dim3(threads), 0, stream, tokens, (const TW*)table, (const TW*)pair, scale, mul_prev, \
+            mul_cur, buckets, prev, out, H, V, positions, row_req, req_row_start, req_n_rows, req_state_slot, writes)
+  if (dtype == KF_F32) KF_GO(float);
+  else if (dtype == KF_BF16) KF_GO(__nv_bfloat16);
+  else return KF_ERR_DTYPE;
+#undef KF_GO
+  KF_CHECK_LAUNCH();
+  return KF_OK;
+}
+
 // cos/sin of position * inv_freq[i], all in 32-bit (accurate sincosf: no fast-math in this library).
 // The product of a position and a 32-bit frequency has up to 48 significant bits; rounded to 32-bit it is off by up to
 // 2.4e-4 rad at position 4,000, which a 32-bit engine with scores of 40 shows in its logits.  So the product is kept as

@@ -48,6 +48,7 @@ struct Pool {
 struct Group {
   int keep = 0;                          // tokens at the start of a request that stay readable behind the window
   int window;                            // -1: none
+  bool chunked = false;                  // `window` is the size of chunks counted from position 0, not a sliding window
   Pool pool;
   std::vector<int> mirror;               // [max_requests][width]: block tables by state slot, -1 where no page
   Group(int w, int n_pages) : window(w), pool(n_pages) {}
@@ -193,6 +194,14 @@ KF_HOST_API int kf_cache_keep_first(void* h, int g, int keep) {
   return OK;
 }
 
+// group g's requests read only the chunk their newest token stands in (chunks of the group's window size)
+KF_HOST_API int kf_cache_chunked(void* h, int g) {
+  Cache* c = (Cache*)h;
+  if (g < 0 || g >= (int)c->groups.size() || c->groups[g].window < 1) return E_COMMIT;
+  c->groups[g].chunked = true;
+  return OK;
+}
+
 // the step that wrote n_new reserved tokens succeeded: advance, and give back the pages a window has passed
 KF_HOST_API int kf_cache_commit(void* h, int64_t req, int n_new) {
   Cache* c = (Cache*)h;
@@ -205,8 +214,9 @@ KF_HOST_API int kf_cache_commit(void* h, int64_t req, int n_new) {
   for (size_t g = 0; g < c->groups.size(); ++g) {
     const int w = c->groups[g].window;
     if (w < 0) continue;
-    // a query at position p reads keys >= p - w + 1; the next query sits at r.length
-    const int dead = std::min(std::max(0, r.length - w + 1) / c->page_size, r.n_entries[g]);
+    // a query at position p reads keys >= p - w + 1, or from its chunk's first position on; the next query sits at r.length
+    const int first = c->groups[g].chunked ? r.length / w * w : std::max(0, r.length - w + 1);
+    const int dead = std::min(first / c->page_size, r.n_entries[g]);
     int* row = c->row((int)g, r.slot);
     const int kept = (c->groups[g].keep + c->page_size - 1) / c->page_size;       // pages of the kept first tokens stay
     for (int i = std::max(r.first_live[g], kept); i < dead; ++i) {

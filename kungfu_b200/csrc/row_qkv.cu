@@ -8,6 +8,8 @@
 //   `interleaved`, else (i, i + rot/2); cos and sin are multiplied by `mag`
 //   value mixing: vmode 1 writes the biased v of the row to v_shared [T, nkv * dv] (32-bit); vmode 2 replaces v by
 //   (1 - lambda) v + lambda v_shared[t] (lambda: one number on the device); what was mixed is what is filed
+//   v_at: the column (from col0) v starts at, nq + nk for a v of its own, nq where the keys as projected (biased, before norm and
+//   rotation) are the values too; its bias stands at the same place
 //   q goes to q_out [T, nh * D], k and v to the token's place in the request's pages; heads use D elements, tails zero.
 // kf_cols_rmsnorm: out[t, i] = in[t, c0 + i] / sqrt(mean_i(in[t, c0 + i]^2) + eps) * w[i] for a column range of a 32-bit
 //   matrix (the normed latent a second projection reads).
@@ -19,7 +21,7 @@ __global__ void __launch_bounds__(256)
 rownorm_rope_append_kernel(const float* __restrict__ in, int ld, int col0, const TW* __restrict__ bias,
                            const TW* __restrict__ wq, const TW* __restrict__ wk, float eps, const float* __restrict__ cos_t,
                            const float* __restrict__ sin_t, int rot, int interleaved, float mag, int nh, int nkv, int dk,
-                           int dv, int D, const TW* __restrict__ lambda, float* __restrict__ v_shared, int vmode,
+                           int dv, int D, int v_at, const TW* __restrict__ lambda, float* __restrict__ v_shared, int vmode,
                            const int* __restrict__ positions, const int* __restrict__ row_req,
                            const int* __restrict__ block_table, int table_stride, int page_size, TKV* __restrict__ pages,
                            TQ* __restrict__ q_out, int write_kv, int T) {
@@ -84,7 +86,7 @@ rownorm_rope_append_kernel(const float* __restrict__ in, int ld, int col0, const
     float y = 0.f;
     if (e < dv) {
       const int j = head * dv + e;
-      y = src[nq + nk + j] + (bias ? kf_load(bias, nq + nk + j) : 0.f);
+      y = src[v_at + j] + (bias ? kf_load(bias, v_at + j) : 0.f);
       if (vmode == 1) v_shared[(size_t)t * nv + j] = y;
       else if (vmode == 2) y = (1.f - lam) * y + lam * v_shared[(size_t)t * nv + j];
     }
@@ -94,7 +96,7 @@ rownorm_rope_append_kernel(const float* __restrict__ in, int ld, int col0, const
 
 KF_API int kf_rownorm_rope_append(const float* in, int ld, int col0, const void* bias, const void* wq, const void* wk,
                                   int w_dtype, float eps, const float* cos_t, const float* sin_t, int rot, int interleaved,
-                                  float mag, int nh, int nkv, int dk, int dv, int D, const void* lambda, float* v_shared,
+                                  float mag, int nh, int nkv, int dk, int dv, int D, int v_at, const void* lambda, float* v_shared,
                                   int vmode, const int* positions, const int* row_req, const int* block_table,
                                   int table_stride, int page_size, void* pages, int kv_dtype, void* q_out, int q_dtype,
                                   int write_kv, int T, cudaStream_t stream) {
@@ -102,6 +104,7 @@ KF_API int kf_rownorm_rope_append(const float* in, int ld, int col0, const void*
   if (dk > D || dv > D || dk < 1 || dv < 1 || rot > dk || (rot & 1) || nkv < 1 || nh % nkv) return KF_ERR_SIZE;
   if (rot > 0 && (!cos_t || !sin_t)) return KF_ERR_SIZE;
   if (vmode != 0 && !v_shared) return KF_ERR_SIZE;
+  if (v_at < 0 || col0 + v_at + nkv * dv > ld) return KF_ERR_SIZE;
   const size_t smem = (size_t)(nh + nkv) * dk * sizeof(float);
   if (smem > 200 * 1024) return KF_ERR_SIZE;
 #define KF_GO(TW, TQ, TKV)                                                                                              \
@@ -109,7 +112,7 @@ KF_API int kf_rownorm_rope_append(const float* in, int ld, int col0, const void*
     if (smem > 48 * 1024)                                                                                               \
       cudaFuncSetAttribute(rownorm_rope_append_kernel<TW, TQ, TKV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
     kf_launch(rownorm_rope_append_kernel<TW, TQ, TKV>, dim3(T), dim3(256), smem, stream, in, ld, col0, (const TW*)bias,  \
-              (const TW*)wq, (const TW*)wk, eps, cos_t, sin_t, rot, interleaved, mag, nh, nkv, dk, dv, D,              \
+              (const TW*)wq, (const TW*)wk, eps, cos_t, sin_t, rot, interleaved, mag, nh, nkv, dk, dv, D, v_at,        \
               (const TW*)lambda, v_shared, vmode, positions, row_req, block_table, table_stride, page_size,            \
               (TKV*)pages, (TQ*)q_out, write_kv, T);                                                                    \
   } while (0)

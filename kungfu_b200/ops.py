@@ -473,7 +473,8 @@ def linear_rope_kv_append(x, wqkv, cos, sin, rot: int, n_heads: int, n_kv_heads:
 
 @_dispatch("paged_attention")
 def paged_attention(q, out, ctx, cache, n_heads: int, n_kv_heads: int, head_dim: int, scale: float, softcap: float,
-                    window: int | None, value_split: int = 0, keep_first: int = 0, sink: bool = False) -> None:
+                    window: int | None, value_split: int = 0, keep_first: int = 0, sink: bool = False,
+                    chunk: int | None = None, sigmoid_bias=None) -> None:
     """Causal (optionally windowed, softcapped) attention of every row of the step over its request's pages.
     bfloat16: rows of single-row requests run the split-KV decode kernel, the rest the prefill kernel, when the
     head size has an instance of them; the 32-bit path and other head sizes run the generic kernel.
@@ -481,18 +482,28 @@ def paged_attention(q, out, ctx, cache, n_heads: int, n_kv_heads: int, head_dim:
     the pages G heads (n_kv_heads = G * G counts (key head, value head) pairs): result head h, of pair p = h // r with
     r = n_heads // n_kv_heads, is query head (p // G) * r + h % r over the keys of head p // G and the values of head p % G.
     keep_first = K > 0 (with a window): keys 0..K-1 stay visible behind the window, at their true positions.
-    sink: one is added to the softmax's denominator (a key of score 0 that has no value)."""
+    sink: one is added to the softmax's denominator (a key of score 0 that has no value).
+    chunk = C (instead of a window): key j is seen from position p iff j <= p and j // C == p // C.
+    sigmoid_bias (32-bit, one number per head): no softmax; key j counts with sigmoid(s_j + sigmoid_bias[h]), and the
+    weights are not normalized."""
     T = q.shape[0]
+    if chunk and window:
+        raise KernelError("paged_attention: a window or chunks, not both")
+    if sigmoid_bias is not None and (sink or value_split or sigmoid_bias.dtype != torch.float32 or sigmoid_bias.numel() != n_heads):
+        raise KernelError("paged_attention: sigmoid weights take one 32-bit number per head, no sink and no value split")
+    if chunk and value_split:
+        raise KernelError("paged_attention: chunks with a value split are not supported")
     keep_first = int(keep_first) if window else 0
-    extras = (keep_first, int(bool(sink)))
+    reach = int(chunk) if chunk else (int(window) if window else 0)      # the most keys a row can see (0: no bound)
+    extras = (keep_first, int(bool(sink)), _p(sigmoid_bias))
     lib = library()
     table = ctx.block_tables[cache.group]
     pages = cache.pages
     common = (_p(ctx.positions), _p(ctx.row_req), _p(table), table.shape[1], cache.page_size, n_heads, n_kv_heads, head_dim,
-              _f(scale), _f(softcap), int(window or 0), int(value_split))
+              _f(scale), _f(softcap), -int(chunk) if chunk else int(window or 0), int(value_split))
     n_dec = getattr(ctx, "n_dec_rows", 0)
     fast = (use_fast_attention and q.dtype == torch.bfloat16 and pages.dtype == torch.bfloat16)
-    if (keep_first or sink) and (value_split or not extras_on_fast_kernels or not decode_on_tensor_cores
+    if (keep_first or sink or sigmoid_bias is not None) and (value_split or not extras_on_fast_kernels or not decode_on_tensor_cores
                                or n_heads // n_kv_heads > 16):
         fast = False                                   # the generic kernel: every combination
     vs_splits = ctypes.c_int(0)
@@ -514,7 +525,7 @@ def paged_attention(q, out, ctx, cache, n_heads: int, n_kv_heads: int, head_dim:
         rest, n_rest = ctx.pre_rows, ctx.n_pre_rows
     elif fast and n_dec > 0 and lib.kf_attention_decode_supported(head_dim):
         ht, splits = ctypes.c_int(0), ctypes.c_int(0)
-        max_keys = min(ctx.max_kv_len, window + keep_first) if window else ctx.max_kv_len
+        max_keys = min(ctx.max_kv_len, reach + keep_first) if reach else ctx.max_kv_len
         group = n_heads // n_kv_heads
         if decode_on_tensor_cores and group <= 16:
             lib.kf_attention_decode_mma_plan(n_dec, n_heads, n_kv_heads, head_dim, int(max_keys), ctypes.byref(splits))
@@ -541,7 +552,7 @@ def paged_attention(q, out, ctx, cache, n_heads: int, n_kv_heads: int, head_dim:
     if (prompt_tiles and prefill_on_tcgen05 and getattr(ctx, "n_wide", 0) > 0
             and lib.kf_attention_prefill_tc_supported(head_dim, cache.page_size, _p(q), _p(pages))):
         sc = _dev_scratch(q.device)
-        max_keys = min(ctx.max_kv_len, window + 128 + -(-keep_first // 64) * 64) if window else ctx.max_kv_len
+        max_keys = min(ctx.max_kv_len, reach + 128 + -(-keep_first // 64) * 64) if reach else ctx.max_kv_len
         run_tiles = ctypes.c_int(0)
         if prefill_plan_override is not None:
             parts, run_tiles = int(prefill_plan_override[0]), ctypes.c_int(int(prefill_plan_override[1]))
@@ -892,27 +903,118 @@ def cols_rmsnorm(x, c0: int, weight, eps: float, out) -> None:
 @_dispatch("rownorm_rope_append")
 def rownorm_rope_append(proj, col0: int, bias, q_norm, k_norm, eps: float, cos, sin, rot: int, interleaved: bool,
                         magnitude: float, n_heads: int, n_kv_heads: int, key_dim: int, value_dim: int, ctx, cache, q_out,
-                        v_mix=None, v_shared=None, v_mode: int = 0) -> None:
+                        v_mix=None, v_shared=None, v_mode: int = 0, values_are_keys: bool = False) -> None:
     """From the 32-bit [q | k | v] columns of `proj` to the attention's operands: optional bias, RMS norm of q and of k
     over ALL their heads at once (weights of n_heads * key_dim and n_kv_heads * key_dim; None: no norm), rotation of the
     first `rot` elements of every head (interleaved pairs or halves), q into `q_out` [T, n_heads * D], k and v into the
     pages of `cache`.  v_mode 1: the biased v is also written to `v_shared` [T, n_kv_heads * value_dim] (32-bit);
-    v_mode 2: v <- (1 - v_mix) v + v_mix v_shared before it is filed (`v_mix`: one number on the device)."""
+    v_mode 2: v <- (1 - v_mix) v + v_mix v_shared before it is filed (`v_mix`: one number on the device).
+    values_are_keys: `proj` has no v columns; the keys as projected (biased, before norm and rotation) are filed as values."""
     T = q_out.shape[0]
     D = cache.pages.shape[-1]
     if q_out.shape[1] != n_heads * D:
         raise KernelError(f"rownorm_rope_append: q rows of {q_out.shape[1]} elements for {n_heads} heads of {D}")
     table = ctx.block_tables[cache.group]
+    v_at = (n_heads if values_are_keys else n_heads + n_kv_heads) * key_dim
     ws = [w for w in (bias, q_norm, k_norm, v_mix) if w is not None]
     wdt = _dt(ws[0]) if ws else _dt(q_out)
     if any(_dt(w) != wdt for w in ws):
         raise KernelError("rownorm_rope_append: bias, norm weights and the mixing number must share one element type")
     _check(library().kf_rownorm_rope_append(_p(proj), proj.shape[1], int(col0), _p(bias), _p(q_norm), _p(k_norm), wdt, _f(eps),
                                             _p(cos), _p(sin), int(rot), int(bool(interleaved)), _f(magnitude), n_heads,
-                                            n_kv_heads, key_dim, value_dim, D, _p(v_mix), _p(v_shared), int(v_mode),
+                                            n_kv_heads, key_dim, value_dim, D, v_at, _p(v_mix), _p(v_shared), int(v_mode),
                                             _p(ctx.positions), _p(ctx.row_req), _p(table), table.shape[1], cache.page_size,
                                             _p(cache.pages), _dt(cache.pages), _p(q_out), _dt(q_out), int(cache.writes), T,
                                             _stream()), "rownorm_rope_append")
+
+
+@_dispatch("embed_pair")
+def embed_pair(tokens, table, pair, scale: float, mul_prev: int, mul_cur: int, prev, out, ctx, writes: bool = True) -> None:
+    """out[t, :] = table[tokens[t], :] * scale + pair[row, :], row = (previous token * mul_prev + token * mul_cur) mod
+    buckets with buckets = pair's rows - 1, and the last row for a request's first token (32-bit out).  `prev` [slots, 1]
+    int32: the last token of every live request; read for a request's first row of the step and moved on."""
+    T, (V, H) = out.shape[0], table.shape
+    if pair.dtype != table.dtype or pair.shape[1] != H or pair.shape[0] < 2:
+        raise KernelError(f"embed_pair: tables {tuple(table.shape)} {table.dtype} and {tuple(pair.shape)} {pair.dtype} do not agree")
+    L = ctypes.c_longlong
+    _check(library().kf_embed_pair(_p(tokens), _p(table), _p(pair), _dt(table), _f(scale), L(mul_prev), L(mul_cur),
+                                   L(pair.shape[0] - 1), _p(prev), _p(out), T, H, V, _p(ctx.positions), _p(ctx.row_req),
+                                   _p(ctx.req_row_start), _p(ctx.req_n_rows), _p(ctx.req_state_slot), int(writes), _stream()),
+           "embed_pair")
+
+
+@_dispatch("input_conv")
+def input_conv(x, weight, state, out, ctx, writes: bool = True) -> None:
+    """out[t] = x[t] + sum_j weight[:, j] x_(t - taps + 1 + j) over the rows of every request of the step (32-bit x, out in
+    the weights' element type); rows before the step come from `state` [slots, taps - 1, width] (32-bit; None when taps
+    is 1), which is moved on in the same launch."""
+    T, W = x.shape
+    _check(library().kf_input_conv(_p(x), _p(weight), _dt(weight), W, int(weight.shape[1]), _p(state), _p(out), _dt(out),
+                                   _p(ctx.row_req), _p(ctx.req_row_start), _p(ctx.req_n_rows), _p(ctx.req_state_slot), T,
+                                   int(writes), _stream()), "input_conv")
+
+
+@_dispatch("add_rmsnorm_conv")
+def add_rmsnorm_conv(branch, weight, eps: float, residual, conv_weight, state, out, ctx, writes: bool = True) -> bool:
+    """residual += rmsnorm(branch) * weight, then out = the convolution of `input_conv` of the new residual: one launch for
+    steps in which no request has more than one row.  True if it ran; False if its sizes have no instance (then the
+    caller runs `add_rmsnorm` and `input_conv`)."""
+    T, H = residual.shape
+    lib = library()
+    if weight.dtype != conv_weight.dtype or not lib.kf_add_rmsnorm_conv_supported(H, int(conv_weight.shape[1])):
+        return False
+    _check(lib.kf_add_rmsnorm_conv(_p(branch), _p(weight), _p(conv_weight), _dt(weight), _f(eps), _p(residual),
+                                   int(conv_weight.shape[1]), _p(state), _p(out), _dt(out), _p(ctx.row_req),
+                                   _p(ctx.req_state_slot), T, H, int(writes), _stream()), "add_rmsnorm_conv")
+    return True
+
+
+DECAY_CHUNK_ROWS = 256       # rows per chunk when a step's chunks are walked side by side
+DECAY_CHUNKED_FROM = 512     # rows of a step from which they are ...
+DECAY_CHUNKED_BLOCKS = 296   # ... if walking whole requests would take at most this many blocks (two per SM)
+decay_chunks = True          # False: every request's rows are walked from its state to its state by one block per tile
+
+
+def decay_powers(decay) -> torch.Tensor:
+    """[heads, DECAY_CHUNK_ROWS + 1]: decay_h^0, decay_h^1, ..., made in 64-bit."""
+    a = torch.tensor([float(x) for x in decay], dtype=torch.float64)
+    return torch.pow(a[:, None], torch.arange(DECAY_CHUNK_ROWS + 1, dtype=torch.float64)[None, :]).to(torch.float32).contiguous()
+
+
+def decay_memory_takes_bfloat16(dim: int, vdim: int, ld: int) -> bool:
+    """Whether prompt portions of these sizes run on the tensor cores from bfloat16 rows of `ld` columns."""
+    if _override is not None:
+        return False
+    return bool(use_tensor_cores and library().kf_decay_chunk_supported(int(dim), int(vdim), int(ld)))
+
+
+@_dispatch("decay_memory")
+def decay_memory(rows, q0: int, k0: int, v0: int, act, powers, state, out, heads: int, dim: int, vdim: int, ctx,
+                 writes: bool = True) -> None:
+    """S <- a_h S + k v^T, o = S^T q over the rows of every request of the step, from and into `state`
+    [slots, heads, dim, vdim] (32-bit); a_h = powers[h, 1] (`decay_powers`).  q, k, v are column ranges of `rows`, laid out
+    head by head: 32-bit (act 'silu' is applied to them as they are read) or bfloat16 that has been through it (act
+    None).  out: 32-bit [rows, heads * vdim].  bfloat16 rows of prompt portions run on the tensor cores; a long step with
+    few heads and requests is cut into chunks that are walked side by side (three launches)."""
+    T = out.shape[0]
+    lib = library()
+    if act not in (None, "silu"):
+        raise KernelError(f"decay_memory: activation {act!r} is not one of None, silu")
+    single = bool(getattr(ctx, "decode_only", False))
+    chunk_rows = n_numbers = 0
+    chunk_state = None
+    if (rows.dtype == torch.bfloat16 and not single and decay_chunks and T >= DECAY_CHUNKED_FROM
+            and ctx.n_reqs * heads * lib.kf_decay_chunk_tiles(dim, vdim) <= DECAY_CHUNKED_BLOCKS
+            and lib.kf_decay_chunk_supported(dim, vdim, rows.shape[1])):
+        chunk_rows = DECAY_CHUNK_ROWS
+        n_numbers = T // chunk_rows + ctx.n_reqs
+        chunk_state = ctx.buf("decay_chunk_state", (n_numbers, heads, dim, vdim), torch.float32)
+    _check(lib.kf_decay_memory(_p(rows), _dt(rows), rows.shape[1], int(q0), int(k0), int(v0), int(act == "silu"), _p(powers),
+                               powers.shape[1], _p(state), _p(out), heads, dim, vdim, ctx.n_reqs, _p(ctx.req_row_start),
+                               _p(ctx.req_n_rows), _p(ctx.req_state_slot), int(writes), int(single), chunk_rows, n_numbers,
+                               _p(chunk_state), _stream()), "decay_memory")
+    if chunk_rows:
+        add_launches(2)
 
 
 MLSTM_COLUMNS = 16          # value columns a block of the matrix memory's walk owns

@@ -4,15 +4,16 @@ from .base import (Block, FeedForward, FixedState, Mixer, Norm, PagedKV, Part, P
                    register_position)
 from .norm import GroupRmsNorm, NoNorm, RmsNorm
 from .rope import Rope
-from .conv import ShortConv
+from .conv import InputConv, ShortConv
 from .attention import ConvGatedAttention, PagedAttention, RowNormAttention, TalkingAttention
 from .ssm import Mamba2Mixer
 from .latent import LatentAttention
 from .delta import GatedDeltaMixer
+from .lightning import LightningAttention
 from .mlstm import MatrixMemory, SideBySide
 from .moe import RoutedExperts
 from .side import TokenSide
 from .ffn import DenseFfn, GatedFfn, PolyNormFfn
-from .embedding import Embedding, LmHead
+from .embedding import Embedding, LmHead, PairEmbedding
 from .block import ParallelBlock, SandwichBlock, ScaledBlock
 from .model import DecoderModel, LayerCall, default_schedule

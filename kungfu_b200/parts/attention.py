@@ -249,8 +249,11 @@ class RowNormAttention(Mixer):
       v <- (1 - lambda) v + lambda v_first                      `v_mix` "mix": v_first = the biased v of the same token in
                                                                  the layer whose `v_mix` is "first" and whose `v_mix_tag`
                                                                  is the same; the mixed v is what the pages hold
-      s_j = (q . k_j) * scale; key j is seen from position p iff j <= p and (no window, or p - j < window, or j < keep_first)
-      a = exp(s_j) / (sum exp(s) + 1 if `sink` else sum exp(s))
+      `values_are_keys`: there is no v in the projection; the keys as projected (biased, before norm and rotation) are v
+      s_j = (q . k_j) * scale; key j is seen from position p iff j <= p and (no window, or p - j < window, or j < keep_first);
+                                                                 with `chunk` C instead: j <= p and j // C == p // C
+      a = exp(s_j) / (sum exp(s) + 1 if `sink` else sum exp(s));  with `sigmoid_bias` instead: a = sigmoid(s_j + bias_h),
+                                                                 not normalized over the keys
       o_h <- o_h * sigmoid(g_h)                                  one gate per head, from the same input x (`gated`)
       y = o W_o^T
     Scores, softmax, norms, rotation, mixing and gate are 32-bit."""
@@ -260,7 +263,14 @@ class RowNormAttention(Mixer):
                  position: PositionEncoding | None = None, bias: torch.Tensor | None = None,
                  q_norm: torch.Tensor | None = None, k_norm: torch.Tensor | None = None, norm_eps: float = 1e-6,
                  gated: bool = False, v_mix: str | None = None, v_mix_weight: torch.Tensor | None = None,
-                 v_mix_tag: str = "v_first", out_tag: str = "branch_out"):
+                 v_mix_tag: str = "v_first", out_tag: str = "branch_out", values_are_keys: bool = False,
+                 chunk: int | None = None, sigmoid_bias: torch.Tensor | None = None):
+        if values_are_keys and key_dim != value_dim:
+            raise ValueError(f"keys of {key_dim} cannot be values of {value_dim}")
+        if chunk is not None and window is not None:
+            raise ValueError("a mixer has a window or chunks, not both")
+        if sigmoid_bias is not None and sink:
+            raise ValueError("the sink is a term of a softmax's denominator; sigmoid weights have none")
         if n_heads % n_kv_heads:
             raise ValueError(f"n_heads {n_heads} is not a multiple of n_kv_heads {n_kv_heads}")
         if v_mix not in (None, "first", "mix"):
@@ -280,7 +290,11 @@ class RowNormAttention(Mixer):
         self.v_mix_weight = v_mix_weight.reshape(-1).contiguous() if (v_mix_weight is not None and v_mix_weight.numel()) else None
         if v_mix == "mix" and self.v_mix_weight is None and (v_mix_weight is None):
             raise ValueError("v_mix 'mix' needs the mixing number")
-        self.qkv_width = (self.n_heads + self.n_kv_heads) * self.key_dim + self.n_kv_heads * self.value_dim
+        self.values_are_keys = bool(values_are_keys)
+        self.chunk = None if chunk is None else int(chunk)
+        self.sigmoid_bias = None if sigmoid_bias is None else sigmoid_bias.to(torch.float32).contiguous()
+        self.qkv_width = (self.n_heads + self.n_kv_heads) * self.key_dim
+        self.qkv_width += 0 if self.values_are_keys else self.n_kv_heads * self.value_dim
         self.proj_width = self.qkv_width + (self.n_heads if self.gated else 0)
         self.width = wo.shape[0]
         if w_in.numel() and w_in.shape[0] != self.proj_width:
@@ -293,7 +307,7 @@ class RowNormAttention(Mixer):
         ops.check_attention_sizes(self.n_heads, self.n_kv_heads, self.head_dim)
 
     def state_need(self):
-        return PagedKV(self.n_kv_heads, self.head_dim, self.window, self.keep_first)
+        return PagedKV(self.n_kv_heads, self.head_dim, self.window, self.keep_first, self.chunk)
 
     def forward(self, x, ctx, cache):
         proj = ctx.buf("attn_proj", (x.shape[0], self.proj_width), torch.float32)
@@ -326,10 +340,11 @@ class RowNormAttention(Mixer):
             mode = 1 if self.v_mix == "first" else 2
         ops.rownorm_rope_append(proj, col0, self.bias, self.q_norm, self.k_norm, self.norm_eps, cos, sin, rot, interleaved, mag,
                                 nh, nkv, self.key_dim, self.value_dim, ctx, cache, q,
-                                v_mix=self.v_mix_weight if mode == 2 else None, v_shared=shared, v_mode=mode)
+                                v_mix=self.v_mix_weight if mode == 2 else None, v_shared=shared, v_mode=mode,
+                                values_are_keys=self.values_are_keys)
         o = ctx.buf("attn_o", (T, nh * D), ctx.act_dtype)
         ops.paged_attention(q, o, ctx, cache, nh, nkv, D, self.scale, 0.0, self.window, keep_first=self.keep_first,
-                            sink=self.sink)
+                            sink=self.sink, chunk=self.chunk, sigmoid_bias=self.sigmoid_bias)
         if heads_out is not None:                      # the gated heads, times `scale`, into a row another product reads
             ops.head_gate(o, proj if self.gated else None, col0 + self.qkv_width, nh, self.value_dim, D, heads_out, ctx,
                           out_col0=out_col0, scale=scale)

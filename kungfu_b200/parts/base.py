@@ -26,11 +26,13 @@ import torch
 @dataclass(frozen=True)
 class PagedKV:
     """Keys and values for every past token, in pages; `window` keys at most are ever read when set, plus the first
-    `keep_first` tokens of the request, which stay readable behind the window."""
+    `keep_first` tokens of the request, which stay readable behind the window.  `chunk`, when set (instead of a window):
+    only keys of the reader's own run of `chunk` positions, counted from the request's start, are ever read."""
     n_kv_heads: int
     head_dim: int
     window: int | None = None
     keep_first: int = 0
+    chunk: int | None = None
 
 
 @dataclass(frozen=True)
@@ -145,6 +147,16 @@ class Block(Part):
     """An arrangement of norms, one mixer and one feed-forward around the residual stream."""
 
     mixer: Mixer
+
+    def state_need(self) -> StateNeed | None:
+        """What this block's cache slot holds per request: its mixer's state (a block with a state of its own adds it)."""
+        return self.mixer.state_need()
+
+    def first_step(self, cache):
+        """The norm this block starts with, for the block before it to fuse into its last kernel (`cache`: this block's
+        cache view, for a first step that keeps a state)."""
+        return self.pre_mixer
+
     # A block that sets this takes forward(x, ctx, cache, normed=None, then=None) and returns (x, normed_for_next):
     # `normed` is its own first norm computed by the block before it, `then` the next block's first norm.
     fuses_next_norm = False

@@ -4,13 +4,16 @@
 `Residual` with a post norm, two of them per block, gemma2.rs:39-41):
   h   = x + post_mixer(mixer(pre_mixer(x)))
   out = h + post_ffn(ffn(pre_ffn(h)))
+`pre_mixer` may be an input convolution (`InputConv`) instead of a norm: the mixer then reads the convolved stream, and the
+block's cache slot holds the convolution's state behind the mixer's.
 A post norm of None gives the plain pre-norm block other models use; `ffn` None a layer of the first line alone.
 The residual stream and its sums stay in 32-bit.
 """
 from __future__ import annotations
 
 from .. import ops
-from .base import Block, FeedForward, Mixer, Norm, register_block
+from .base import Block, FeedForward, Mixer, Norm, StateBundle, register_block
+from .conv import InputConv
 from .norm import RmsNorm
 
 
@@ -24,10 +27,33 @@ class SandwichBlock(Block):
         self.pre_mixer, self.mixer, self.post_mixer = pre_mixer, mixer, post_mixer
         self.pre_ffn, self.ffn, self.post_ffn = pre_ffn, ffn, post_ffn
 
+    def _conv_need(self):
+        return self.pre_mixer.state_need() if isinstance(self.pre_mixer, InputConv) else None
+
+    def state_need(self):
+        need, conv = self.mixer.state_need(), self._conv_need()
+        if conv is None:
+            return need
+        return conv if need is None else StateBundle((need, conv))
+
+    def _views(self, cache):
+        """(what the mixer is given, the input convolution's view) of this block's cache view."""
+        if self._conv_need() is None:
+            return cache, None
+        need = self.mixer.state_need()
+        if need is None:
+            return None, cache
+        return (cache[:-1] if isinstance(need, StateBundle) else cache[0]), cache[-1]
+
+    def first_step(self, cache):
+        if isinstance(self.pre_mixer, InputConv):
+            return self.pre_mixer.bind(self._views(cache)[1])
+        return self.pre_mixer
+
     def forward(self, x, ctx, cache, normed=None, then=None):
         act = ctx.act_dtype
-        n = normed if normed is not None else self.pre_mixer.forward(x, ctx, act)
-        a = self.mixer.forward(n, ctx, cache)
+        n = normed if normed is not None else self.first_step(cache).forward(x, ctx, act)
+        a = self.mixer.forward(n, ctx, self._views(cache)[0])
         if self.ffn is None:                                   # a layer without a feed-forward
             if self.post_mixer is not None:
                 return x, self.post_mixer.add_into(a, x, ctx, then=then, out_dtype=act if then is not None else None)

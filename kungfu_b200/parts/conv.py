@@ -14,7 +14,7 @@ from __future__ import annotations
 import torch
 
 from .. import ops
-from .base import FixedState, Part
+from .base import FixedState, Norm, Part
 
 
 class ShortConv(Part):
@@ -46,3 +46,37 @@ class ShortConv(Part):
         if state_view.writes:
             ops.short_conv_commit(proj, col0, in_bias, self.channels, self.taps, state_view.state, ctx,
                                   w_dtype=self.weight.dtype)
+
+
+class InputConv(Part):
+    """What a sublayer reads is replaced by h + conv(h): a causal convolution over time of the residual stream, one filter
+    per channel, added to its own input.  It stands in a block's place of the norm before the mixer (`SandwichBlock`);
+    the block's cache slot then also holds its state, the last taps - 1 inputs in 32-bit."""
+
+    def __init__(self, weight: torch.Tensor):
+        self.weight = weight                            # [width, taps]; the last column multiplies the current token
+        self.width, self.taps = int(weight.shape[0]), int(weight.shape[1]) if weight.dim() == 2 else 1
+        if not (1 <= self.taps <= 8):
+            raise ValueError(f"an input convolution has 1 to 8 taps, found {self.taps}")
+
+    def state_need(self):
+        return FixedState((self.taps - 1, self.width), torch.float32) if self.taps > 1 else None
+
+    def bind(self, view) -> "BoundInputConv":
+        return BoundInputConv(self, view)
+
+
+class BoundInputConv(Norm):
+    """An input convolution with the cache view of one call: what a block's first step looks like to the block before it."""
+
+    def __init__(self, conv: InputConv, view):
+        self.conv, self.width = conv, conv.width
+        self.state = view.state if view is not None else None
+        self.writes = view.writes if view is not None else True
+
+    def forward(self, x, ctx, out_dtype, rows=None):
+        if rows is not None:
+            raise NotImplementedError("an input convolution runs over whole steps only")
+        out = ctx.buf("norm_out", (x.shape[0], self.width), out_dtype)
+        ops.input_conv(x, self.conv.weight, self.state, out, ctx, writes=self.writes)
+        return out

@@ -19,7 +19,9 @@ Options for other models of the kind:
                       dot product is added to the score: s = (q_h . W_uk,h c + q_rot,h . k_rot) * scale.  In the latent
                       space the shared part simply rides behind c in the stored key row (zeros in the value row) and
                       behind W_uk,h^T q_h in the query.
-  `w_gate`            head h's result is multiplied by sigmoid(W_g x)_h before the output projection.
+  `window`            key j is seen from position p iff 0 <= p - j < window
+  `w_gate`            head h's result is multiplied by sigmoid(W_g x)_h before the output projection (W_g: one row per
+                      head), or, with `gate_elements`, every element of the concatenated heads by its own (H * dv rows).
 """
 from __future__ import annotations
 
@@ -68,7 +70,7 @@ class LatentAttention(Mixer):
                  wo: torch.Tensor, *, n_heads: int, dim: int, vdim: int, rank: int, scale: float, norm_eps: float,
                  window: int | None = None, w_dq: torch.Tensor | None = None, dq_norm: torch.Tensor | None = None,
                  rot_dim: int = 0, position: PositionEncoding | None = None, w_gate: torch.Tensor | None = None,
-                 out_tag: str = "branch_out"):
+                 gate_elements: bool = False, out_tag: str = "branch_out"):
         self.n_heads, self.dim, self.vdim, self.rank = int(n_heads), int(dim), int(vdim), int(rank)
         self.rot_dim = int(rot_dim) if position is not None else 0
         self.position = position
@@ -78,7 +80,7 @@ class LatentAttention(Mixer):
         self.width = wo.shape[0]
         self.c_norm, self.wo, self.dq_norm, self.out_tag = c_norm, wo, dq_norm, out_tag
         self.q_latent = w_dq is not None
-        self.gated = w_gate is not None
+        self.gated, self.gate_elements = w_gate is not None, bool(gate_elements)
         H, d, dv, r, rd = self.n_heads, self.dim, self.vdim, self.rank, self.rot_dim
         self.q_rank = int(w_dq.shape[0]) if (self.q_latent and w_dq.numel()) else 0
         given = [w_q, w_dkv, w_uk, w_uv] + ([w_dq] if self.q_latent else []) + ([w_gate] if self.gated else [])
@@ -102,7 +104,10 @@ class LatentAttention(Mixer):
         self.q_width = H * (d + rd)
         self.c_col = self.q_rank if self.q_latent else self.q_width
         self.g_col = self.c_col + r + rd
-        self.proj_width = max(self.g_col + (H if self.gated else 0), self.w_in.shape[0])
+        gate_rows = (H * dv if self.gate_elements else H) if self.gated else 0
+        if self.gated and w_gate.numel() and w_gate.shape[0] != gate_rows:
+            raise ValueError(f"the gate has {w_gate.shape[0]} rows, expected {gate_rows}")
+        self.proj_width = max(self.g_col + gate_rows, self.w_in.shape[0])
         ops.check_attention_sizes(H, 1, D, largest=_KERNEL_HEAD_SIZES[-1])
 
     def state_need(self):
@@ -142,7 +147,10 @@ class LatentAttention(Mixer):
         ops.head_linear(o, 0, self.w_uv, v)
         if self.gated:
             gated = ctx.buf("attn_gated", (T, H * self.vdim), ctx.act_dtype)
-            ops.head_gate(v, proj, self.g_col, H, self.vdim, self.vdim, gated, ctx)
+            if self.gate_elements:
+                ops.head_mix_gate(v, None, proj, self.g_col, H, H, self.vdim, self.vdim, gated, ctx)
+            else:
+                ops.head_gate(v, proj, self.g_col, H, self.vdim, self.vdim, gated, ctx)
             v = gated
         y = ctx.buf(self.out_tag, (T, self.width), torch.float32)
         ops.linear(v, self.wo, y)

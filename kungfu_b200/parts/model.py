@@ -52,18 +52,21 @@ class DecoderModel(Part):
         if sorted(writers) != list(range(len(writers))):
             raise ValueError("cache slots must be numbered 0..n-1")
         self._writers = writers
+        self._embedding_keeps = getattr(embedding, "state_need", lambda: None)() is not None
 
     def children(self):
         return [self.embedding, *self.layers, self.head]
 
     def state_needs(self) -> list[StateNeed | None]:
-        """Per cache slot, what the mixer that writes it keeps per request."""
-        return [self.layers[self._writers[s]].mixer.state_need() for s in range(len(self._writers))]
+        """Per cache slot, what the block that writes it keeps per request; the last slot is the embedding's, if it keeps
+        something (the token before)."""
+        needs = [self.layers[self._writers[s]].state_need() for s in range(len(self._writers))]
+        return needs + ([self.embedding.state_need()] if self._embedding_keeps else [])
 
     def forward(self, ctx):
         """Runs exactly the rows in `ctx`; returns 32-bit logits for `ctx.logit_rows` (None if none wanted)."""
         with ops.nvtx_range("embedding"):
-            x = self.embedding.forward(ctx)
+            x = self.embedding.forward(ctx, ctx.cache_view(len(self._writers), True)) if self._embedding_keeps else self.embedding.forward(ctx)
         normed = None
         for i, call in enumerate(self.schedule):
             block = self.layers[call.layer]
@@ -81,7 +84,9 @@ class DecoderModel(Part):
                     # nothing is added to the residual in between
                     nxt_call = self.schedule[i + 1] if i + 1 < len(self.schedule) else None
                     nxt = self.layers[nxt_call.layer] if nxt_call is not None and nxt_call.shift is None else None
-                    then = nxt.pre_mixer if nxt is not None and getattr(nxt, "fuses_next_norm", False) else None
+                    then = None
+                    if nxt is not None and getattr(nxt, "fuses_next_norm", False):
+                        then = nxt.first_step(ctx.cache_view(nxt_call.cache, nxt_call.writes))
                     x, normed = block.forward(x, ctx, view, normed=normed, then=then)
                 else:
                     x, normed = block.forward(x, ctx, view), None

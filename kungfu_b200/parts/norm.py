@@ -11,6 +11,7 @@ import torch
 
 from .. import ops
 from .base import Norm, register_norm
+from .conv import BoundInputConv
 
 
 class RmsNorm(Norm):
@@ -26,8 +27,19 @@ class RmsNorm(Norm):
         ops.rmsnorm(x, self.weight, self.eps, self.plus_one, out, rows)
         return out
 
+    def scaled(self, factor: float) -> "RmsNorm":
+        """The same norm with its result multiplied by `factor` (in its 32-bit weights)."""
+        w = self.weight.to(torch.float32) + (1.0 if self.plus_one else 0.0)
+        return RmsNorm(w * float(factor), self.eps)
+
     def add_into(self, branch, residual, ctx, then=None, out_dtype=None):
-        """residual += norm(branch); returns then(residual) if `then` is given (one kernel when `then` is an RmsNorm)."""
+        """residual += norm(branch); returns then(residual) if `then` is given (one kernel when `then` is an RmsNorm, or, in
+        a step of single rows, the next block's input convolution)."""
+        if isinstance(then, BoundInputConv) and not self.plus_one and getattr(ctx, "decode_only", False):
+            out = ctx.buf("norm_out", (residual.shape[0], self.width), out_dtype)
+            if ops.add_rmsnorm_conv(branch, self.weight, self.eps, residual, then.conv.weight, then.state, out, ctx,
+                                    writes=then.writes):
+                return out
         if then is None:
             ops.add_rmsnorm(branch, self.weight, self.eps, self.plus_one, residual)
             return None

@@ -64,6 +64,9 @@ def _register_builtin() -> None:
     from .config.nukelix import NukelixConfig
     from .models import nukelix
     register("Nukelix", NukelixConfig.from_dict, nukelix.build, nukelix.tensor_specs, replace=True)
+    from .config.lurisun import LurisunConfig
+    from .models import lurisun
+    register("Lurisun", LurisunConfig.from_dict, lurisun.build, lurisun.tensor_specs, replace=True)
 
 
 _register_builtin()
