@@ -9,6 +9,7 @@
     python bench.py --compare petanex
     python bench.py --compare pimodra
     python bench.py --compare nukelix
+    python bench.py --compare lurisun
                     (Bolonex beside Gemma 2, or Petanex beside Bolonex, at equal layer sizes: prefill and decode throughput
                     and, per operation, the time of one step against the time its bytes, or its multiply-adds, take at the
                     measured rates; one JSON line)
@@ -800,6 +801,66 @@ def compare_nukelix(args) -> dict:
                                                                       ("petanex", petanex_config(z), petanex_op_bytes)))
 
 
+# ---- Lurisun beside Nukelix at equal layer sizes (--compare lurisun) ---------------------------------------------------
+# Eight layers in both.  Lurisun: latent attention, linear attention with fixed decays, sigmoid attention over chunks, linear
+# attention, twice; every feed-forward dense.  Nukelix (the closest existing model: blocks that read the residual stream,
+# row-normed attention, attention over a latent with queries through their own, a 32-bit memory with a d x dv state per
+# head) as in --compare nukelix.  Same width, heads, head size, state size per head, latents, reach of the attention and
+# vocabulary; Nukelix's chosen and shared experts together have the dense feed-forward's width.
+LURISUN_SIZES = {name: dict(z) for name, z in NUKELIX_SIZES.items()}
+
+
+def lurisun_config(z: dict) -> dict:
+    d, h = z["dim"], z["d_heads"]
+    att = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": d, "vdim": d, "scale": d ** -0.5, "mask": {"size": z["window"]},
+           "rot": {"base": 500000.0, "dims": d // 2}}
+    lig = {"heads": h, "dim": z["d_dim"], "vdim": z["d_vdim"], "decay": [1.0 - 2.0 ** -(2.0 + 6.0 * i / h) for i in range(h)]}
+    lat = {"heads": z["lat_heads"], "dim": d, "vdim": d, "kv_rank": z["kv_rank"], "q_rank": z["q_rank"], "scale": d ** -0.5,
+           "mask": {"size": z["window"]}}
+    kinds = ["latent_attention", "lightning", "attention", "lightning"]
+    layers = [{"type": kinds[i % 4], "mixer": (lat, lig, att, lig)[i % 4], "mlp": {"kind": "dense", "ff": z["ff"]}}
+              for i in range(COMPARE_LAYERS)]
+    return {"architecture": "Lurisun", "width": z["width"], "vocab": COMPARE_VOCAB, "norm": {"eps": 1e-6}, "logit_scale": 1.0,
+            "canon": {"taps": 4}, "embedding": {"bigram": {"mul_prev": 31, "mul_cur": 17, "buckets": COMPARE_VOCAB}}, "layers": layers}
+
+
+def lurisun_op_bytes(z: dict, T: int, n_reqs: int, keys: int) -> dict:
+    """Bytes (and, for the products, floating-point operations) each operation of one Lurisun step must move, summed over
+    the layers that use it; a prompt's attention also has the multiply-adds of the keys its rows see."""
+    W, H, G, d, L = z["width"], z["heads"], z["kv_heads"], z["dim"], COMPARE_LAYERS
+    n_att, n_lat, n_lig = L // 4, L // 4, L // 2
+    mh, md, mv = z["d_heads"], z["d_dim"], z["d_vdim"]
+    lh, rank = z["lat_heads"], z["kv_rank"]
+    D = 256 if rank > 128 else 128
+    seen = min(keys, z["window"])
+    single = T == n_reqs
+    cq = (H + G) * d
+    # query-key pairs of a prompt: chunks of `window`, and a sliding window
+    pairs_c = sum(i % z["window"] + 1 for i in range(T)) if not single else n_reqs * seen
+    pairs_w = sum(min(i + 1, z["window"]) for i in range(T)) if not single else n_reqs * seen
+    return {
+        "embed_pair": T * W * 8,
+        "input_conv": L * T * W * 6,
+        "add_rmsnorm_conv": L * T * W * 14,
+        "rownorm_rope_append": n_att * T * (4 * cq + 2 * (cq + G * d) + 4 * d),
+        "paged_attention": (n_att * (n_reqs * seen * 2 * G * d * 2 + T * H * d * 4) + n_lat * (n_reqs * seen * 2 * D * 2 + T * lh * D * 4),
+                            n_att * 4 * H * d * pairs_c + n_lat * 4 * lh * D * pairs_w),
+        "decay_memory": n_lig * (T * mh * (2 * md + mv) * (4 if single else 2) + T * mh * mv * 4 + 2 * n_reqs * mh * md * mv * 4),
+        "head_norm_gate": n_lig * T * mh * mv * 10,
+        "latent_append": n_lat * T * (rank * 4 + 4 * D),
+        "cols_rmsnorm": n_lat * T * z["q_rank"] * 6,
+        "head_linear": (n_lat * T * lh * (4 * d + 2 * D + 2 * D + 2 * d), n_lat * 4 * T * lh * D * d),
+        "element_gate": n_lat * T * lh * d * 8,
+        "add_rmsnorm": (L if single else 2 * L) * T * W * 14,
+        "linear_gated": (L * (2 * z["ff"] * W * 2 + T * (2 * W + 2 * z["ff"])), L * 4 * T * z["ff"] * W),
+    }
+
+
+def compare_lurisun(args) -> dict:
+    return compare_models(args, "lurisun", LURISUN_SIZES, lambda z: (("lurisun", lurisun_config(z), lurisun_op_bytes),
+                                                                      ("nukelix", nukelix_config(z), nukelix_op_bytes)))
+
+
 def micro_attention() -> int:
     """Decode attention alone: eight launches over distinct pages replayed from a CUDA graph, per batch size; one JSON
     line each with microseconds per launch and bytes of keys and values over that time."""
@@ -1254,15 +1315,15 @@ def main() -> int:
     ap.add_argument("--only-headline", action="store_true", help="skip the other batch sizes, the mixed steps, 32-bit and the other model sizes")
     ap.add_argument("--micro", choices=["attention", "prompt-attention", "gemm", "products", "qkv-rope", "reference", "memory"],
                     help="time kernels alone instead of the model step")
-    ap.add_argument("--compare", choices=["bolonex", "petanex", "pimodra", "nukelix"],
-                    help="another workload: Bolonex beside Gemma 2, Petanex beside Bolonex, or Pimodra beside Gemma 2, at equal "
+    ap.add_argument("--compare", choices=["bolonex", "petanex", "pimodra", "nukelix", "lurisun"],
+                    help="another workload: Bolonex beside Gemma 2, Petanex beside Bolonex, Pimodra beside Gemma 2, Nukelix beside Petanex, or Lurisun beside Nukelix, at equal "
                          "layer sizes (prefill, decode, per-operation rooflines)")
     args = ap.parse_args()
     if args.compare:
         args.warmup = max(args.warmup, 3)
         args.reps = max(args.reps, 1)
         print(json.dumps({"bolonex": compare_bolonex, "petanex": compare_petanex, "pimodra": compare_pimodra,
-                          "nukelix": compare_nukelix}[args.compare](args)))
+                          "nukelix": compare_nukelix, "lurisun": compare_lurisun}[args.compare](args)))
         return 0
     if args.micro:
         return {"attention": micro_attention, "prompt-attention": micro_prompt_attention, "gemm": micro_gemm,

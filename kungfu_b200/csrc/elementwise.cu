@@ -87,6 +87,43 @@ KF_API int kf_embed_pair(const int* tokens, const void* table, const void* pair,
   return KF_OK;
 }
 
+// out[t, i] = x[t, i] * sigmoid(gate[t, col0 + i]), gate a wider 32-bit matrix: one gate per element.  VEC = 4 where rows and
+// columns start on four elements.
+template <typename T, int VEC>
+__global__ void element_gate_kernel(const T* __restrict__ x, const float* __restrict__ gate, int ld, int col0, T* __restrict__ out,
+                                    int n_rows, int n) {
+  kf_pdl_trigger();
+  kf_pdl_wait();
+  const long i = ((long)blockIdx.x * blockDim.x + threadIdx.x) * VEC;
+  if (i >= (long)n_rows * n) return;
+  const int t = (int)(i / n), c = (int)(i - (long)t * n);
+  const float* g = gate + (size_t)t * ld + col0 + c;
+  float z[VEC], v[VEC];
+  if constexpr (VEC == 4) {
+    const float4 q = *reinterpret_cast<const float4*>(g);
+    z[0] = q.x, z[1] = q.y, z[2] = q.z, z[3] = q.w;
+  } else z[0] = g[0];
+#pragma unroll
+  for (int k = 0; k < VEC; ++k) v[k] = kf_load(x, (size_t)i + k) / (1.f + expf(-z[k]));
+#pragma unroll
+  for (int k = 0; k < VEC; ++k) kf_store(out, (size_t)i + k, v[k]);
+}
+
+KF_API int kf_element_gate(const void* x, const float* gate, int ld, int col0, void* out, int dtype, int n_rows, int n,
+                           cudaStream_t stream) {
+  if (n_rows <= 0 || n <= 0) return KF_OK;
+  if (col0 < 0 || col0 + n > ld) return KF_ERR_SIZE;
+  const bool vec = n % 4 == 0 && ld % 4 == 0 && col0 % 4 == 0 && (((uintptr_t)x | (uintptr_t)gate | (uintptr_t)out) & 15) == 0;
+  const int grid = kf_ceil_div((long)n_rows * n, 256 * (vec ? 4 : 1));
+#define KF_GO(T, VEC) kf_launch(element_gate_kernel<T, VEC>, dim3(grid), dim3(256), 0, stream, (const T*)x, gate, ld, col0, (T*)out, n_rows, n)
+  if (dtype == KF_F32) { if (vec) KF_GO(float, 4); else KF_GO(float, 1); }
+  else if (dtype == KF_BF16) { if (vec) KF_GO(__nv_bfloat16, 4); else KF_GO(__nv_bfloat16, 1); }
+  else return KF_ERR_DTYPE;
+#undef KF_GO
+  KF_CHECK_LAUNCH();
+  return KF_OK;
+}
+
 // cos/sin of position * inv_freq[i], all in 32-bit (accurate sincosf: no fast-math in this library).
 // The product of a position and a 32-bit frequency has up to 48 significant bits; rounded to 32-bit it is off by up to
 // 2.4e-4 rad at position 4,000, which a 32-bit engine with scores of 40 shows in its logits.  So the product is kept as

@@ -943,6 +943,15 @@ def embed_pair(tokens, table, pair, scale: float, mul_prev: int, mul_cur: int, p
            "embed_pair")
 
 
+@_dispatch("element_gate")
+def element_gate(x, gate, col0: int, out) -> None:
+    """out[t, i] = x[t, i] * sigmoid(gate[t, col0 + i]); x and out of one element type, gate 32-bit and as wide as it is."""
+    T, n = out.shape
+    if tuple(x.shape) != (T, n) or x.dtype != out.dtype:
+        raise KernelError(f"element_gate: x{tuple(x.shape)} {x.dtype} and out{tuple(out.shape)} {out.dtype} do not agree")
+    _check(library().kf_element_gate(_p(x), _p(gate), gate.shape[1], int(col0), _p(out), _dt(out), T, n, _stream()), "element_gate")
+
+
 @_dispatch("input_conv")
 def input_conv(x, weight, state, out, ctx, writes: bool = True) -> None:
     """out[t] = x[t] + sum_j weight[:, j] x_(t - taps + 1 + j) over the rows of every request of the step (32-bit x, out in

@@ -148,7 +148,7 @@ class LatentAttention(Mixer):
         if self.gated:
             gated = ctx.buf("attn_gated", (T, H * self.vdim), ctx.act_dtype)
             if self.gate_elements:
-                ops.head_mix_gate(v, None, proj, self.g_col, H, H, self.vdim, self.vdim, gated, ctx)
+                ops.element_gate(v, proj, self.g_col, gated)
             else:
                 ops.head_gate(v, proj, self.g_col, H, self.vdim, self.vdim, gated, ctx)
             v = gated

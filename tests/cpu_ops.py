@@ -99,7 +99,8 @@ class CpuOps:
             cache.pages[page, 0, :, pos % P, :] = k[t].to(cache.pages.dtype)
             cache.pages[page, 1, :, pos % P, :] = v[t].to(cache.pages.dtype)
 
-    def paged_attention(self, q, out, ctx, cache, nh, nkv, d, scale, softcap, window, value_split=0, keep_first=0, sink=False):
+    def paged_attention(self, q, out, ctx, cache, nh, nkv, d, scale, softcap, window, value_split=0, keep_first=0, sink=False,
+                        chunk=None, sigmoid_bias=None):
         T = q.shape[0]
         table = ctx.block_tables[cache.group]
         P = cache.page_size
@@ -111,7 +112,7 @@ class CpuOps:
                 out[t] = 0
                 continue
             pos = int(ctx.positions[t])
-            lo = max(0, pos - window + 1) if window else 0
+            lo = max(0, pos - window + 1) if window else (pos // chunk * chunk if chunk else 0)
             js = list(range(0, min(keep_first, lo) if window else 0)) + list(range(lo, pos + 1))
             pages = [int(table[r, j // P]) for j in js]
             assert all(p >= 0 for p in pages), f"row {t} reads a page that was given back"
@@ -129,7 +130,9 @@ class CpuOps:
                 s = (K[:, kh] @ qt[qh]) * scale
                 if softcap > 0:
                     s = softcap * torch.tanh(s / softcap)
-                if sink:                      # one more term, exp(0), in the denominator
+                if sigmoid_bias is not None:
+                    p = torch.sigmoid(s + sigmoid_bias[h])
+                elif sink:                    # one more term, exp(0), in the denominator
                     p = torch.softmax(torch.cat([s, s.new_zeros(1)]), dim=0)[:-1]
                 else:
                     p = torch.softmax(s, dim=0)
@@ -452,14 +455,14 @@ class CpuOps:
             y[..., rot // 2:rot] = b * c + a * s_
 
     def rownorm_rope_append(self, proj, col0, bias, q_norm, k_norm, eps, cos, sin, rot, interleaved, magnitude, nh, nkv, dk, dv,
-                            ctx, cache, q_out, v_mix=None, v_shared=None, v_mode=0):
+                            ctx, cache, q_out, v_mix=None, v_shared=None, v_mode=0, values_are_keys=False):
         T = q_out.shape[0]
         D = cache.pages.shape[-1]
-        C = (nh + nkv) * dk + nkv * dv
+        C = (nh + nkv) * dk + (0 if values_are_keys else nkv * dv)
         x = proj[:T, col0:col0 + C].float()
         if bias is not None:
             x = x + bias.float()[None, :]
-        q, k, v = x[:, :nh * dk].clone(), x[:, nh * dk:(nh + nkv) * dk].clone(), x[:, (nh + nkv) * dk:].clone()
+        q, k, v = x[:, :nh * dk].clone(), x[:, nh * dk:(nh + nkv) * dk].clone(), x[:, (nh if values_are_keys else nh + nkv) * dk:].clone()
         if q_norm is not None:
             q = q * torch.rsqrt(q.pow(2).mean(-1, keepdim=True) + eps) * q_norm.float()
         if k_norm is not None:
@@ -549,6 +552,60 @@ class CpuOps:
                 memory[slot] = S
                 norm_state[slot, :, :m_at] = nn.repeat(1, m_at // d)
                 norm_state[slot, :, m_at] = m
+
+    # ---- an embedding of token pairs, convolved inputs, decayed linear attention ----------------------------------------
+    @staticmethod
+    def _requests(ctx):
+        """(request, its rows of the step, its state slot) for every request that has rows."""
+        for r in range(ctx.n_reqs):
+            n, slot = int(ctx.req_n_rows[r]), int(ctx.req_state_slot[r])
+            if n > 0 and slot >= 0:
+                yield r, range(int(ctx.req_row_start[r]), int(ctx.req_row_start[r]) + n), slot
+
+    def embed_pair(self, tokens, table, pair, scale, mul_prev, mul_cur, prev, out, ctx, writes=True):
+        out.zero_()
+        for _, rows, slot in self._requests(ctx):
+            before = int(prev[slot, 0])
+            for t in rows:
+                tok = int(tokens[t])
+                b = pair.shape[0] - 1
+                row = b if int(ctx.positions[t]) == 0 else (before * mul_prev + tok * mul_cur) % b
+                out[t] = table[tok].float() * scale + pair[row].float()
+                before = tok
+            if writes:
+                prev[slot, 0] = before
+
+    def element_gate(self, x, gate, col0, out):
+        out.copy_((x.float() * torch.sigmoid(gate[:x.shape[0], col0:col0 + x.shape[1]])).to(out.dtype))
+
+    def input_conv(self, x, weight, state, out, ctx, writes=True):
+        taps = weight.shape[1]
+        for _, rows, slot in self._requests(ctx):
+            past = [state[slot, s].clone() for s in range(taps - 1)] if taps > 1 else []
+            for t in rows:
+                past.append(x[t].clone())
+                y = x[t] + sum(weight[:, j].float() * past[len(past) - taps + j] for j in range(taps))
+                out[t] = y.to(out.dtype)
+            if writes and taps > 1:
+                for s in range(taps - 1):
+                    state[slot, s] = past[len(past) - (taps - 1) + s]
+
+    def add_rmsnorm_conv(self, branch, weight, eps, residual, conv_weight, state, out, ctx, writes=True):
+        return False                                   # the caller runs add_rmsnorm and input_conv
+
+    def decay_memory(self, rows, q0, k0, v0, act, powers, state, out, heads, dim, vdim, ctx, writes=True):
+        f = (lambda t: t * torch.sigmoid(t)) if act == "silu" else (lambda t: t)
+        a = powers[:, 1][:, None, None]
+        for _, mine, slot in self._requests(ctx):
+            S = state[slot].clone()
+            for t in mine:
+                q = f(rows[t, q0:q0 + heads * dim].float()).view(heads, dim)
+                k = f(rows[t, k0:k0 + heads * dim].float()).view(heads, dim)
+                v = f(rows[t, v0:v0 + heads * vdim].float()).view(heads, vdim)
+                S = a * S + k[:, :, None] * v[:, None, :]
+                out[t] = (S * q[:, :, None]).sum(1).reshape(-1)
+            if writes:
+                state[slot] = S
 
     def weighted_sum2(self, a, sa, b, sb, out):
         out.copy_(sa * a + sb * b)

@@ -177,10 +177,20 @@ def latent_attention(h, w, p: str, m: dict, eps: float):
     cq = rms(linear(h, w[p + "dq"]), eps) * w[p + "dq.norm"].to(F)
     q = linear(cq, w[p + "uq"]).view(T, H, d)
     c = rms(linear(h, w[p + "dkv"]), eps) * w[p + "dkv.norm"].to(F)
-    k = linear(c, w[p + "uk"]).view(T, H, d)
-    v = linear(c, w[p + "uv"]).view(T, H, dv)
     mask = window_mask(T, m["mask"]["size"] if m.get("mask") else None)
-    o = softmax_attend(q, k, v, m["scale"], mask).reshape(T, H * dv)
+    if ROUND is _EXACT:
+        k = linear(c, w[p + "uk"]).view(T, H, d)
+        v = linear(c, w[p + "uv"]).view(T, H, dv)
+        o = softmax_attend(q, k, v, m["scale"], mask)
+    else:
+        # the same attention in the latent space, as a path that caches c alone has to: q . (U c) = (U^T q) . c, and the
+        # values' map applied after the weighted sum.  Exactly equal; what is rounded differs.
+        uk, uv = w[p + "uk"].to(F).view(H, d, -1), w[p + "uv"].to(F).view(H, dv, -1)
+        ql = torch.einsum("thd,hdr->thr", ROUND(q), uk)
+        cs = c[:, None, :].expand(T, H, c.shape[-1])
+        ol = ROUND(softmax_attend(ql, cs, cs, m["scale"], mask))
+        o = torch.einsum("thr,hvr->thv", ol, uv)
+    o = o.reshape(T, H * dv)
     return linear(o * sigmoid(linear(h, w[p + "g"])), w[p + "o"])
 
 
