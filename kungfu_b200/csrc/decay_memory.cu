@@ -182,7 +182,6 @@ __global__ void __launch_bounds__(LANES * DW_COLS) decay_walk_kernel(DecayArgs p
 // ---- 64 rows at a time on the tensor cores -----------------------------------------------------------------------------
 
 constexpr int DC_ROWS = 64;
-constexpr int DC_WARPS = 4;
 enum { DC_WHOLE = 0, DC_STATES = 1, DC_FROM_STATES = 2 };
 
 // The chunk a block walks: chunks of `chunk_rows` rows are numbered request by request (requests without rows have none).
@@ -203,17 +202,23 @@ __device__ __forceinline__ void dc_split(float x, float y, uint32_t* hi, uint32_
   *lo = kf_mma::pack_bf16(x - f.x, y - f.y);
 }
 
-// D: the key size rounded up to a size with an instance (tails zero); VT: value columns per block.
+// D: the key size rounded up to a size with an instance (tails zero); VT: value columns per block; WARPS: 4 or 8 (eight keep
+// the parts of a 256-row state in registers; below that four are the faster ones, having less to recompute).
 // mode DC_WHOLE: from and into the request's state.  DC_STATES: every chunk but a request's last, from zero, no results, into
 // chunk_state[number].  DC_FROM_STATES: from chunk_state[number]; a request's last chunk into its state.
-template <int D, int VT>
-__global__ void __launch_bounds__(DC_WARPS * 32)
+template <int D, int VT, int WARPS>
+__global__ void __launch_bounds__(WARPS * 32)
 decay_chunk_kernel(DecayArgs p, int mode, int chunk_rows, float* __restrict__ chunk_state) {
   using namespace kf_mma;
   kf_pdl_trigger();
   constexpr int KS = D / 16;                           // k-steps along the key size
-  constexpr int MT = D / 64;                           // 16-row tiles of the state per warp
   constexpr int NT = VT / 8;                           // 8-column tiles of the values
+  // The state: RG groups of rows x CG groups of columns, one per warp.  The results: four tiles of 16 rows x OG groups of
+  // columns (the warps of a row tile all compute its scores).
+  constexpr int RG = (WARPS == 8 && D >= 128) ? 8 : 4, CG = WARPS / RG, OG = WARPS / 4;
+  constexpr int MT = D / RG / 16;                      // 16-row tiles of the state per warp
+  constexpr int NTS = NT / CG;                         // ... and its 8-column tiles
+  constexpr int NTO = NT / OG;                         // 8-column tiles of the results per warp
   constexpr int QK_TILE = DC_ROWS * D, V_TILE = DC_ROWS * VT;
   extern __shared__ __align__(128) uint8_t dc_smem[];
   __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(dc_smem);         // [2][64][D]
@@ -236,7 +241,9 @@ decay_chunk_kernel(DecayArgs p, int mode, int chunk_rows, float* __restrict__ ch
   const int n = min(chunk_rows, p.n_rows[req] - chunk * chunk_rows);
   const int col0 = tile * VT;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
-  for (int i = tid; i <= DC_ROWS; i += DC_WARPS * 32) pw[i] = p.powers[(size_t)h * p.n_powers + i];
+  const int wr = warp & 3, oc = (warp >> 2) * NTO;     // this warp's tile of rows, its first column tile of the results
+  const int sr = (warp % RG) * (D / RG), sc = (warp / RG) * NTS;   // its first row and first column tile of the state
+  for (int i = tid; i <= DC_ROWS; i += WARPS * 32) pw[i] = p.powers[(size_t)h * p.n_powers + i];
   kf_pdl_wait();
 
   const __nv_bfloat16* qg = kf_produced((const __nv_bfloat16*)p.q) + h * p.d;
@@ -246,7 +253,7 @@ decay_chunk_kernel(DecayArgs p, int mode, int chunk_rows, float* __restrict__ ch
   auto load = [&](int c0, int st) {
     constexpr int CH = D / 8, CV = VT / 8;
     const int rows = n - c0;
-    for (int i = tid; i < DC_ROWS * CH; i += DC_WARPS * 32) {
+    for (int i = tid; i < DC_ROWS * CH; i += WARPS * 32) {
       const int t = i / CH, c = i - t * CH;
       const bool ok = t < rows && c * 8 < p.d;
       const size_t row = (size_t)(first + c0 + (ok ? t : 0));
@@ -254,7 +261,7 @@ decay_chunk_kernel(DecayArgs p, int mode, int chunk_rows, float* __restrict__ ch
       cp_async16(tile_ptr<D>(sK + st * QK_TILE, t, c), kg + row * p.ldk + cc, ok);
       if (with_out) cp_async16(tile_ptr<D>(sQ + st * QK_TILE, t, c), qg + row * p.ldq + cc, ok);
     }
-    for (int i = tid; i < DC_ROWS * CV; i += DC_WARPS * 32) {
+    for (int i = tid; i < DC_ROWS * CV; i += WARPS * 32) {
       const int t = i / CV, c = i - t * CV;
       const bool ok = t < rows && col0 + c * 8 < p.dv;
       const size_t row = (size_t)(first + c0 + (ok ? t : 0));
@@ -264,18 +271,18 @@ decay_chunk_kernel(DecayArgs p, int mode, int chunk_rows, float* __restrict__ ch
   load(0, 0);
   cp_async_commit();
 
-  // this warp's rows of the state: warp * (D / 4) + mt * 16 + {g, g + 8}, columns nt * 8 + tq * 2 + {0, 1}
-  float S[MT][NT][4];
+  // this warp's part of the state: rows sr + mt * 16 + {g, g + 8}, columns (sc + nt) * 8 + tq * 2 + {0, 1}
+  float S[MT][NTS][4];
   float* own = p.state + ((size_t)slot * p.H + h) * p.d * p.dv;
   float* kept = chunk_state + ((size_t)number * p.H + h) * p.d * p.dv;
   const float* from = mode == DC_WHOLE ? own : kept;
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
-    for (int nt = 0; nt < NT; ++nt)
+    for (int nt = 0; nt < NTS; ++nt)
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
-        const int row = warp * (D / 4) + mt * 16 + g + 8 * e, col = col0 + nt * 8 + tq * 2;
+        const int row = sr + mt * 16 + g + 8 * e, col = col0 + (sc + nt) * 8 + tq * 2;
         float2 v = make_float2(0.f, 0.f);
         if (mode != DC_STATES && row < p.d && col < p.dv) v = *reinterpret_cast<const float2*>(from + (size_t)row * p.dv + col);
         S[mt][nt][2 * e] = v.x, S[mt][nt][2 * e + 1] = v.y;
@@ -290,57 +297,57 @@ decay_chunk_kernel(DecayArgs p, int mode, int chunk_rows, float* __restrict__ ch
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
-        for (int nt = 0; nt < NT; ++nt)
+        for (int nt = 0; nt < NTS; ++nt)
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
             uint32_t hi, lo;
             dc_split(S[mt][nt][2 * e], S[mt][nt][2 * e + 1], &hi, &lo);
-            const int row = warp * (D / 4) + mt * 16 + g + 8 * e;
-            reinterpret_cast<uint32_t*>(tile_ptr<VT>(sH, row, nt))[tq] = hi;
-            reinterpret_cast<uint32_t*>(tile_ptr<VT>(sL, row, nt))[tq] = lo;
+            const int row = sr + mt * 16 + g + 8 * e;
+            reinterpret_cast<uint32_t*>(tile_ptr<VT>(sH, row, sc + nt))[tq] = hi;
+            reinterpret_cast<uint32_t*>(tile_ptr<VT>(sL, row, sc + nt))[tq] = lo;
           }
     }
     cp_async_wait<1>();
     __syncthreads();
     __nv_bfloat16* k_s = sK + st * QK_TILE;
     __nv_bfloat16* v_s = sV + st * V_TILE;
-    if (with_out && warp * 16 < rows) {
+    if (with_out && wr * 16 < rows) {
       __nv_bfloat16* q_s = sQ + st * QK_TILE;
-      float O[NT][4], P[DC_ROWS / 8][4];
+      float O[NTO][4], P[DC_ROWS / 8][4];
 #pragma unroll
-      for (int nt = 0; nt < NT; ++nt) O[nt][0] = O[nt][1] = O[nt][2] = O[nt][3] = 0.f;
+      for (int nt = 0; nt < NTO; ++nt) O[nt][0] = O[nt][1] = O[nt][2] = O[nt][3] = 0.f;
 #pragma unroll
       for (int nt = 0; nt < DC_ROWS / 8; ++nt) P[nt][0] = P[nt][1] = P[nt][2] = P[nt][3] = 0.f;
 #pragma unroll
       for (int ks = 0; ks < KS; ++ks) {
         uint32_t a[4];
-        ldmatrix_x4(a, tile_ptr<D>(q_s, warp * 16 + (lane & 15), ks * 2 + (lane >> 4)));
+        ldmatrix_x4(a, tile_ptr<D>(q_s, wr * 16 + (lane & 15), ks * 2 + (lane >> 4)));
 #pragma unroll
-        for (int np = 0; np < NT / 2; ++np) {
+        for (int np = 0; np < NTO / 2; ++np) {
           uint32_t b[4];
-          ldmatrix_x4_trans(b, tile_ptr<VT>(sH, ks * 16 + (lane & 7) + (((lane >> 3) & 1) << 3), np * 2 + (lane >> 4)));
+          ldmatrix_x4_trans(b, tile_ptr<VT>(sH, ks * 16 + (lane & 7) + (((lane >> 3) & 1) << 3), oc + np * 2 + (lane >> 4)));
           mma_bf16(O[2 * np], a, b[0], b[1]);
           mma_bf16(O[2 * np + 1], a, b[2], b[3]);
-          ldmatrix_x4_trans(b, tile_ptr<VT>(sL, ks * 16 + (lane & 7) + (((lane >> 3) & 1) << 3), np * 2 + (lane >> 4)));
+          ldmatrix_x4_trans(b, tile_ptr<VT>(sL, ks * 16 + (lane & 7) + (((lane >> 3) & 1) << 3), oc + np * 2 + (lane >> 4)));
           mma_bf16(O[2 * np], a, b[0], b[1]);
           mma_bf16(O[2 * np + 1], a, b[2], b[3]);
         }
 #pragma unroll
         for (int np = 0; np < DC_ROWS / 16; ++np) {
-          if (np > warp) continue;                     // keys after every row of this warp
+          if (np > wr) continue;                     // keys after every row of this warp
           uint32_t b[4];
           ldmatrix_x4(b, tile_ptr<D>(k_s, np * 16 + (lane & 7) + ((lane >> 4) << 3), ks * 2 + ((lane >> 3) & 1)));
           mma_bf16(P[2 * np], a, b[0], b[1]);
           mma_bf16(P[2 * np + 1], a, b[2], b[3]);
         }
       }
-      const int i0 = warp * 16 + g;
+      const int i0 = wr * 16 + g;
       const float d0 = pw[i0 + 1], d1 = pw[i0 + 9];
 #pragma unroll
-      for (int nt = 0; nt < NT; ++nt) { O[nt][0] *= d0; O[nt][1] *= d0; O[nt][2] *= d1; O[nt][3] *= d1; }
+      for (int nt = 0; nt < NTO; ++nt) { O[nt][0] *= d0; O[nt][1] *= d0; O[nt][2] *= d1; O[nt][3] *= d1; }
 #pragma unroll
       for (int nt = 0; nt < DC_ROWS / 8; ++nt) {
-        if (nt > 2 * warp + 1) continue;
+        if (nt > 2 * wr + 1) continue;
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int gap = i0 + 8 * (e >> 1) - (nt * 8 + tq * 2 + (e & 1));
@@ -349,16 +356,16 @@ decay_chunk_kernel(DecayArgs p, int mode, int chunk_rows, float* __restrict__ ch
       }
 #pragma unroll
       for (int ks = 0; ks < DC_ROWS / 16; ++ks) {
-        if (ks > warp) continue;
+        if (ks > wr) continue;
         uint32_t hi[4], lo[4];
         dc_split(P[2 * ks][0], P[2 * ks][1], &hi[0], &lo[0]);
         dc_split(P[2 * ks][2], P[2 * ks][3], &hi[1], &lo[1]);
         dc_split(P[2 * ks + 1][0], P[2 * ks + 1][1], &hi[2], &lo[2]);
         dc_split(P[2 * ks + 1][2], P[2 * ks + 1][3], &hi[3], &lo[3]);
 #pragma unroll
-        for (int np = 0; np < NT / 2; ++np) {
+        for (int np = 0; np < NTO / 2; ++np) {
           uint32_t b[4];
-          ldmatrix_x4_trans(b, tile_ptr<VT>(v_s, ks * 16 + (lane & 7) + (((lane >> 3) & 1) << 3), np * 2 + (lane >> 4)));
+          ldmatrix_x4_trans(b, tile_ptr<VT>(v_s, ks * 16 + (lane & 7) + (((lane >> 3) & 1) << 3), oc + np * 2 + (lane >> 4)));
           mma_bf16(O[2 * np], hi, b[0], b[1]);
           mma_bf16(O[2 * np + 1], hi, b[2], b[3]);
           mma_bf16(O[2 * np], lo, b[0], b[1]);
@@ -366,10 +373,10 @@ decay_chunk_kernel(DecayArgs p, int mode, int chunk_rows, float* __restrict__ ch
         }
       }
 #pragma unroll
-      for (int nt = 0; nt < NT; ++nt)
+      for (int nt = 0; nt < NTO; ++nt)
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
-          const int i = i0 + 8 * e, col = col0 + nt * 8 + tq * 2;
+          const int i = i0 + 8 * e, col = col0 + (oc + nt) * 8 + tq * 2;
           if (i < rows && col < p.dv)
             *reinterpret_cast<float2*>(p.out + (size_t)(first + c0 + i) * p.H * p.dv + h * p.dv + col) =
                 make_float2(O[nt][2 * e], O[nt][2 * e + 1]);
@@ -380,7 +387,7 @@ decay_chunk_kernel(DecayArgs p, int mode, int chunk_rows, float* __restrict__ ch
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
-      for (int nt = 0; nt < NT; ++nt)
+      for (int nt = 0; nt < NTS; ++nt)
 #pragma unroll
         for (int e = 0; e < 4; ++e) S[mt][nt][e] *= dn;
 #pragma unroll
@@ -393,7 +400,7 @@ decay_chunk_kernel(DecayArgs p, int mode, int chunk_rows, float* __restrict__ ch
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt) {
         uint32_t a[4];
-        ldmatrix_x4_trans(a, tile_ptr<D>(k_s, ks * 16 + (lane & 7) + ((lane >> 4) << 3), warp * (D / 32) + mt * 2 + ((lane >> 3) & 1)));
+        ldmatrix_x4_trans(a, tile_ptr<D>(k_s, ks * 16 + (lane & 7) + ((lane >> 4) << 3), sr / 8 + mt * 2 + ((lane >> 3) & 1)));
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const float2 kk = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a[e]));
@@ -401,9 +408,9 @@ decay_chunk_kernel(DecayArgs p, int mode, int chunk_rows, float* __restrict__ ch
         }
       }
 #pragma unroll
-      for (int np = 0; np < NT / 2; ++np) {
+      for (int np = 0; np < NTS / 2; ++np) {
         uint32_t b[4];
-        ldmatrix_x4_trans(b, tile_ptr<VT>(v_s, ks * 16 + (lane & 7) + (((lane >> 3) & 1) << 3), np * 2 + (lane >> 4)));
+        ldmatrix_x4_trans(b, tile_ptr<VT>(v_s, ks * 16 + (lane & 7) + (((lane >> 3) & 1) << 3), sc + np * 2 + (lane >> 4)));
 #pragma unroll
         for (int mt = 0; mt < MT; ++mt) {
           mma_bf16(S[mt][2 * np], hi[mt], b[0], b[1]);
@@ -421,10 +428,10 @@ decay_chunk_kernel(DecayArgs p, int mode, int chunk_rows, float* __restrict__ ch
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
-    for (int nt = 0; nt < NT; ++nt)
+    for (int nt = 0; nt < NTS; ++nt)
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
-        const int row = warp * (D / 4) + mt * 16 + g + 8 * e, col = col0 + nt * 8 + tq * 2;
+        const int row = sr + mt * 16 + g + 8 * e, col = col0 + (sc + nt) * 8 + tq * 2;
         if (row < p.d && col < p.dv)
           *reinterpret_cast<float2*>(to + (size_t)row * p.dv + col) = make_float2(S[mt][nt][2 * e], S[mt][nt][2 * e + 1]);
       }
@@ -464,27 +471,27 @@ decay_chunk_starts_kernel(DecayArgs p, int chunk_rows, float* __restrict__ chunk
   }
 }
 
-template <int D, int VT>
+template <int D, int VT, int WARPS>
 int launch_chunks(const DecayArgs& p, int mode, int chunk_rows, int n_numbers, float* chunk_state, cudaStream_t stream) {
   const size_t smem = (size_t)(4 * DC_ROWS * D + 2 * DC_ROWS * VT + 2 * D * VT) * 2 + (DC_ROWS + 1) * sizeof(float);
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(decay_chunk_kernel<D, VT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+    if (cudaFuncSetAttribute(decay_chunk_kernel<D, VT, WARPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
       kf_record_cuda_error(cudaGetLastError());
       return KF_ERR_SETUP;
     }
     configured = true;
   }
   const dim3 grid((unsigned)((long)n_numbers * p.H * kf_ceil_div(p.dv, VT)));
-  kf_launch(decay_chunk_kernel<D, VT>, grid, dim3(DC_WARPS * 32), smem, stream, p, mode, chunk_rows, chunk_state);
+  kf_launch(decay_chunk_kernel<D, VT, WARPS>, grid, dim3(WARPS * 32), smem, stream, p, mode, chunk_rows, chunk_state);
   KF_CHECK_LAUNCH();
   return KF_OK;
 }
 
 int chunk_pass(const DecayArgs& p, int mode, int chunk_rows, int n_numbers, float* chunk_state, cudaStream_t stream) {
-  if (p.d <= 64) return launch_chunks<64, 64>(p, mode, chunk_rows, n_numbers, chunk_state, stream);
-  if (p.d <= 128) return launch_chunks<128, 64>(p, mode, chunk_rows, n_numbers, chunk_state, stream);
-  return launch_chunks<256, 32>(p, mode, chunk_rows, n_numbers, chunk_state, stream);
+  if (p.d <= 64) return launch_chunks<64, 64, 4>(p, mode, chunk_rows, n_numbers, chunk_state, stream);
+  if (p.d <= 128) return launch_chunks<128, 64, 4>(p, mode, chunk_rows, n_numbers, chunk_state, stream);
+  return launch_chunks<256, 32, 8>(p, mode, chunk_rows, n_numbers, chunk_state, stream);
 }
 
 }  // namespace

@@ -31,6 +31,14 @@ KF_API int kf_embed(const int* tokens, const void* table, int table_dtype, float
   return KF_OK;
 }
 
+__device__ __forceinline__ float4 kf_load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 kf_load4(const __nv_bfloat16* p) {
+  const uint2 r = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+
 // x[t, :] = table[token[t], :] * scale + pair[row(t), :], a second table read by the token and the one before it:
 // row(t) = (previous * mul_prev + token * mul_cur) mod buckets in 64-bit integers, the table's last row (number `buckets`)
 // for a request's first token.  The previous token of a step's first row of a request is its state, prev[slot] (written
@@ -66,6 +74,17 @@ __global__ void embed_pair_kernel(const int* __restrict__ tokens, const TW* __re
   const bool ok = tok >= 0 && tok < V;
   const TW* a = table + (size_t)(ok ? tok : 0) * H;
   const TW* b = pair + (size_t)s_row * H;
+  if ((H & 3) == 0) {                                   // rows start on four elements
+    for (int i = threadIdx.x * 4; i < H; i += blockDim.x * 4) {
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (ok) {
+        const float4 x = kf_load4(a + i), y = kf_load4(b + i);
+        v = make_float4(x.x * scale + y.x, x.y * scale + y.y, x.z * scale + y.z, x.w * scale + y.w);
+      }
+      *reinterpret_cast<float4*>(o + i) = v;
+    }
+    return;
+  }
   for (int i = threadIdx.x; i < H; i += blockDim.x) o[i] = ok ? kf_load(a, i) * scale + kf_load(b, i) : 0.f;
 }
 
@@ -75,6 +94,7 @@ KF_API int kf_embed_pair(const int* tokens, const void* table, const void* pair,
                          int writes, cudaStream_t stream) {
   if (T <= 0) return KF_OK;
   if (buckets < 1 || !prev) return KF_ERR_SIZE;
+  if (H % 4 == 0 && (((uintptr_t)table | (uintptr_t)pair | (uintptr_t)out) & 15)) return KF_ERR_ALIGN;
   const int threads = H >= 1024 ? 256 : 128;
 #define KF_GO(TW)                                                                                                          \
   kf_launch(embed_pair_kernel<TW>, dim3(T), dim3(threads), 0, stream, tokens, (const TW*)table, (const TW*)pair, scale, mul_prev, \

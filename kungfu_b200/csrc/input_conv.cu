@@ -16,6 +16,7 @@
 namespace {
 
 constexpr int IC_MAX_TAPS = 8;
+constexpr int IC_FAST_ROWS = 8;              // rows per block of a long prompt
 
 template <int VEC>
 __device__ __forceinline__ void ic_load(const float* p, float* v) {
@@ -37,6 +38,17 @@ __device__ __forceinline__ void ic_store(__nv_bfloat16* p, const float* v) {
   } else p[0] = __float2bfloat16_rn(v[0]);
 }
 
+__device__ __forceinline__ void ic_load4(const float* p, float* v) {
+  const float4 q = *reinterpret_cast<const float4*>(p);
+  v[0] = q.x, v[1] = q.y, v[2] = q.z, v[3] = q.w;
+}
+__device__ __forceinline__ void ic_load4(const __nv_bfloat16* p, float* v) {
+  const uint2 r = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
+  v[0] = a.x, v[1] = a.y, v[2] = b.x, v[3] = b.y;
+}
+
 // VEC channels per thread, `rows` rows per block; within a run of rows of one request the last taps inputs stay in
 // registers, so every row is read once per block.
 template <typename TW, typename TO, int TAPS, int VEC>
@@ -48,11 +60,20 @@ input_conv_kernel(const float* __restrict__ x, const TW* __restrict__ w, float* 
   const int c0 = (blockIdx.y * blockDim.x + threadIdx.x) * VEC;
   if (c0 >= C) return;
   constexpr int TAIL = TAPS - 1;
-  float wv[VEC][TAPS];
+  constexpr int FAST = TAPS <= 4 ? IC_FAST_ROWS : 0;
+  float wv[VEC][TAPS];                                 // the filters of VEC channels stand one after another
+  if constexpr (VEC == 4) {
+    float flat[4 * TAPS];
 #pragma unroll
-  for (int v = 0; v < VEC; ++v)
+    for (int q = 0; q < TAPS; ++q) ic_load4(w + (size_t)c0 * TAPS + 4 * q, flat + 4 * q);
 #pragma unroll
-    for (int j = 0; j < TAPS; ++j) wv[v][j] = kf_load(w, (size_t)(c0 + v) * TAPS + j);
+    for (int v = 0; v < 4; ++v)
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) wv[v][j] = flat[v * TAPS + j];
+  } else {
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) wv[0][j] = kf_load(w, (size_t)c0 * TAPS + j);
+  }
   kf_pdl_wait();
   x = kf_produced(x);
   float u[TAPS][VEC];                                  // the inputs of the row in hand, oldest first
@@ -73,9 +94,32 @@ input_conv_kernel(const float* __restrict__ x, const TW* __restrict__ w, float* 
 #pragma unroll
       for (int v = 0; v < VEC; ++v) u[j][v] = u[j + 1][v];
   };
-  const int t_end = min(T, (int)(blockIdx.x + 1) * rows);
+  const int t_first = blockIdx.x * rows, t_end = min(T, t_first + rows);
+  // The ordinary block of a long prompt: all its rows belong to one request and see only this step's inputs.  Every load is
+  // then requested before the first sum.
+  if (FAST > 0 && t_end - t_first == FAST && rows == FAST) {
+    const int req = row_req[t_first];
+    if (req >= 0 && row_req[t_end - 1] == req && t_first - req_row_start[req] >= (TAIL > 0 ? TAIL : 1)) {
+      float in[FAST > 0 ? FAST + TAIL : 1][VEC];
+#pragma unroll
+      for (int j = 0; j < FAST + TAIL; ++j) ic_load<VEC>(x + (size_t)(t_first - TAIL + j) * C + c0, in[j]);
+#pragma unroll
+      for (int r = 0; r < FAST; ++r) {
+        float y[VEC];
+#pragma unroll
+        for (int v = 0; v < VEC; ++v) {
+          float acc = 0.f;
+#pragma unroll
+          for (int j = 0; j < TAPS; ++j) acc = fmaf(wv[v][j], in[r + j][v], acc);
+          y[v] = in[r + TAIL][v] + acc;
+        }
+        ic_store<VEC>(out + (size_t)(t_first + r) * C + c0, y);
+      }
+      return;
+    }
+  }
   int held = -2;                                       // the row whose inputs u holds (-2: none)
-  for (int t = blockIdx.x * rows; t < t_end; ++t) {
+  for (int t = t_first; t < t_end; ++t) {
     const int req = row_req[t];
     if (req < 0) { held = -2; continue; }
     const int row0 = req_row_start[req], i = t - row0;
@@ -193,10 +237,10 @@ KF_API int kf_input_conv(const float* x, const void* w, int w_dtype, int C, int 
                          int T, int writes, cudaStream_t stream) {
   if (T <= 0 || C <= 0) return KF_OK;
   if (taps < 1 || taps > IC_MAX_TAPS || (taps > 1 && !state)) return KF_ERR_SIZE;
-  const bool vec = C % 4 == 0 && (((uintptr_t)x | (uintptr_t)state | (uintptr_t)out) & 15) == 0;
+  const bool vec = C % 4 == 0 && (((uintptr_t)x | (uintptr_t)w | (uintptr_t)state | (uintptr_t)out) & 15) == 0;
   const int per_thread = vec ? 4 : 1;
   const int threads = C / per_thread >= 256 ? 256 : 128;
-  const int rows = T >= 2048 ? 16 : (T >= 512 ? 8 : (T >= 64 ? 4 : 1));
+  const int rows = T >= 512 ? IC_FAST_ROWS : (T >= 64 ? 4 : 1);
   const dim3 grid(kf_ceil_div(T, rows), kf_ceil_div(C, threads * per_thread));
 #define KF_LAUNCH(TW, TO, TAPS, VEC)                                                                                  \
   kf_launch(input_conv_kernel<TW, TO, TAPS, VEC>, grid, dim3(threads), 0, stream, x, (const TW*)w, state, (TO*)out, C, row_req, \

@@ -3,6 +3,8 @@
 // kf_latent_append:      c = rms_norm(proj[t, c0 .. c0 + rank)) * w, written into the request's page at the token's
 //                        position, once as the key row and once as the value row of a single key/value head of D >= rank
 //                        elements (tails zero): attention in the latent space reads the same row as key and as value.
+// kf_latent_norms_append: the same, and in the same launch the query latent that stands beside it in the projection:
+//                        cq[t] = rms_norm(proj[t, q0 .. q0 + nq)) * wq, which a second projection reads.
 // kf_latent_rope_append: the same with a rotated key part that all heads share: the r columns after the latent are
 //                        turned by the row's angles (pairs (2i, 2i + 1) when `interleaved`, else (i, i + r/2); cos and sin
 //                        times `mag`) and filed behind c in the key row (the value row holds zeros there); the last r
@@ -57,6 +59,56 @@ __global__ void latent_append_kernel(const float* __restrict__ proj, int ld, int
     kf_store(kdst, i, v);
     kf_store(vdst, i, v);
   }
+}
+
+template <typename TW, typename TC>
+__global__ void __launch_bounds__(256)
+latent_norms_append_kernel(const float* proj, int ld, int q0, int nq, const TW* __restrict__ wq, TC* __restrict__ cq, int c0,
+                           int rank, const TW* __restrict__ w, float eps, const int* __restrict__ positions,
+                           const int* __restrict__ row_req, const int* __restrict__ table, int table_width, int page_size,
+                           TC* __restrict__ pages, int D, int writes) {
+  kf_pdl_trigger();
+  __shared__ float red[33];
+  const int t = blockIdx.x;
+  const int req = row_req[t], pos = positions[t];            // the step's integers: readable at once
+  const int page = req >= 0 ? table[(size_t)req * table_width + pos / page_size] : -1;
+  kf_pdl_wait();
+  proj = kf_produced(proj);
+  const float* a = proj + (size_t)t * ld + q0;
+  const float* c = proj + (size_t)t * ld + c0;
+  float sa = 0.f, sc = 0.f;
+  for (int i = threadIdx.x; i < nq; i += blockDim.x) sa = fmaf(a[i], a[i], sa);
+  for (int i = threadIdx.x; i < rank; i += blockDim.x) sc = fmaf(c[i], c[i], sc);
+  sa = kf_block_sum(sa, red);
+  sc = kf_block_sum(sc, red);
+  const float ia = 1.f / sqrtf(sa / (float)nq + eps), ic = 1.f / sqrtf(sc / (float)rank + eps);
+  for (int i = threadIdx.x; i < nq; i += blockDim.x) kf_store(cq, (size_t)t * nq + i, a[i] * ia * kf_load(wq, i));
+  if (page < 0 || !writes) return;
+  TC* kdst = pages + (((size_t)page * 2 + 0) * page_size + pos % page_size) * D;
+  TC* vdst = pages + (((size_t)page * 2 + 1) * page_size + pos % page_size) * D;
+  for (int i = threadIdx.x; i < D; i += blockDim.x) {
+    const float v = i < rank ? c[i] * ic * kf_load(w, i) : 0.f;
+    kf_store(kdst, i, v);
+    kf_store(vdst, i, v);
+  }
+}
+
+KF_API int kf_latent_norms_append(const float* proj, int ld, int q0, int nq, const void* wq, void* cq, int c0, int rank,
+                                  const void* w, int w_dtype, float eps, const int* positions, const int* row_req,
+                                  const int* table, int table_width, int page_size, void* pages, int dtype, int D, int writes,
+                                  int T, cudaStream_t stream) {
+  if (T <= 0) return KF_OK;
+  if (rank < 1 || rank > D || nq < 1 || q0 < 0 || c0 < 0 || q0 + nq > ld || c0 + rank > ld) return KF_ERR_SIZE;
+#define KF_GO(TW, TC)                                                                                                      \
+  kf_launch(latent_norms_append_kernel<TW, TC>, dim3(T), dim3(nq > 256 ? 256 : 128), 0, stream, proj, ld, q0, nq, (const TW*)wq, \
+            (TC*)cq, c0, rank, (const TW*)w, eps, positions, row_req, table, table_width, page_size, (TC*)pages, D, writes)
+  if (w_dtype == KF_F32 && dtype == KF_F32) KF_GO(float, float);
+  else if (w_dtype == KF_BF16 && dtype == KF_BF16) KF_GO(__nv_bfloat16, __nv_bfloat16);
+  else if (w_dtype == KF_BF16 && dtype == KF_F32) KF_GO(__nv_bfloat16, float);
+  else return KF_ERR_DTYPE;
+#undef KF_GO
+  KF_CHECK_LAUNCH();
+  return KF_OK;
 }
 
 KF_API int kf_latent_append(const float* proj, int ld, int c0, int rank, const void* w, int w_dtype, float eps,

@@ -875,6 +875,20 @@ def latent_append(proj, c0: int, rank: int, weight, eps: float, ctx, cache) -> N
                                       _p(cache.pages), _dt(cache.pages), D, T, _stream()), "latent_append")
 
 
+@_dispatch("latent_norms_append")
+def latent_norms_append(proj, q0: int, q_weight, cq, c0: int, rank: int, weight, eps: float, ctx, cache) -> None:
+    """`latent_append` of columns c0.. and, in the same launch, cq = rms_norm(proj[:, q0:q0 + n]) * q_weight, n = q_weight's
+    length (cq in the pages' element type)."""
+    T, nq = cq.shape
+    table = ctx.block_tables[cache.group]
+    if cq.dtype != cache.pages.dtype or q_weight.dtype != weight.dtype:
+        raise KernelError("latent_norms_append: the two latents must share one element type, and so must their weights")
+    _check(library().kf_latent_norms_append(_p(proj), proj.shape[1], int(q0), nq, _p(q_weight), _p(cq), int(c0), int(rank),
+                                            _p(weight), _dt(weight), _f(eps), _p(ctx.positions), _p(ctx.row_req), _p(table),
+                                            table.shape[1], cache.page_size, _p(cache.pages), _dt(cache.pages),
+                                            cache.pages.shape[-1], int(cache.writes), T, _stream()), "latent_norms_append")
+
+
 @_dispatch("latent_rope_append")
 def latent_rope_append(proj, c0: int, rank: int, rot: int, weight, eps: float, cos, sin, interleaved: bool, magnitude: float,
                        q, q0: int, n_heads: int, q_dim: int, ctx, cache) -> None:
@@ -978,9 +992,9 @@ def add_rmsnorm_conv(branch, weight, eps: float, residual, conv_weight, state, o
     return True
 
 
-DECAY_CHUNK_ROWS = 256       # rows per chunk when a step's chunks are walked side by side
+DECAY_CHUNK_ROWS = 512       # most rows per chunk when a step's chunks are walked side by side
 DECAY_CHUNKED_FROM = 512     # rows of a step from which they are ...
-DECAY_CHUNKED_BLOCKS = 296   # ... if walking whole requests would take at most this many blocks (two per SM)
+DECAY_CHUNKED_BLOCKS = 74    # ... if walking whole requests would take at most this many blocks (half of the SMs)
 decay_chunks = True          # False: every request's rows are walked from its state to its state by one block per tile
 
 
@@ -1015,7 +1029,11 @@ def decay_memory(rows, q0: int, k0: int, v0: int, act, powers, state, out, heads
     if (rows.dtype == torch.bfloat16 and not single and decay_chunks and T >= DECAY_CHUNKED_FROM
             and ctx.n_reqs * heads * lib.kf_decay_chunk_tiles(dim, vdim) <= DECAY_CHUNKED_BLOCKS
             and lib.kf_decay_chunk_supported(dim, vdim, rows.shape[1])):
-        chunk_rows = DECAY_CHUNK_ROWS
+        # chunks of 128, 256 or 512 rows, so that about 256 blocks walk them (measured at 16 and 32 heads x 64 and 128, 2,048
+        # and 8,192 rows: the best of the three is this one)
+        chunk_rows = 128
+        while chunk_rows < DECAY_CHUNK_ROWS and T * heads * lib.kf_decay_chunk_tiles(dim, vdim) >= 512 * chunk_rows:
+            chunk_rows *= 2
         n_numbers = T // chunk_rows + ctx.n_reqs
         chunk_state = ctx.buf("decay_chunk_state", (n_numbers, heads, dim, vdim), torch.float32)
     _check(lib.kf_decay_memory(_p(rows), _dt(rows), rows.shape[1], int(q0), int(k0), int(v0), int(act == "silu"), _p(powers),

@@ -120,7 +120,10 @@ class LatentAttention(Mixer):
         ops.linear(x, self.w_in, proj)
         if self.q_latent:
             cq = ctx.buf("latent_cq", (T, self.q_rank), ctx.act_dtype)
-            ops.cols_rmsnorm(proj, 0, self.dq_norm, self.norm_eps, cq)
+            if self.rot_dim:
+                ops.cols_rmsnorm(proj, 0, self.dq_norm, self.norm_eps, cq)
+            else:                                          # both latents in one launch
+                ops.latent_norms_append(proj, 0, self.dq_norm, cq, self.c_col, self.rank, self.c_norm, self.norm_eps, ctx, cache)
             qf, q0 = ctx.buf("latent_qf", (T, self.q_width), torch.float32), 0
             ops.linear(cq, self.w_uq, qf)
         else:
@@ -130,7 +133,7 @@ class LatentAttention(Mixer):
             ops.latent_rope_append(proj, self.c_col, self.rank, self.rot_dim, self.c_norm, self.norm_eps, cos, sin,
                                    bool(getattr(self.position, "interleaved", False)),
                                    float(getattr(self.position, "magnitude", 1.0)), qf, q0, H, self.dim, ctx, cache)
-        elif cache.writes:
+        elif cache.writes and not self.q_latent:
             ops.latent_append(proj, self.c_col, self.rank, self.c_norm, self.norm_eps, ctx, cache)
         q = ctx.buf("attn_q", (T, H * D), ctx.act_dtype)
         ops.head_linear(qf, q0, self.w_uk_t, q)

@@ -329,6 +329,11 @@ class CpuOps:
             cache.pages[page, 0, 0, pos % cache.page_size] = row.to(cache.pages.dtype)
             cache.pages[page, 1, 0, pos % cache.page_size] = row.to(cache.pages.dtype)
 
+    def latent_norms_append(self, proj, q0, q_weight, cq, c0, rank, weight, eps, ctx, cache):
+        self.cols_rmsnorm(proj, q0, q_weight, eps, cq)
+        if cache.writes:
+            self.latent_append(proj, c0, rank, weight, eps, ctx, cache)
+
     def repeat_rows(self, a, b, parts, out_a, out_b):
         out_a.copy_(a.repeat_interleave(parts))
         out_b.copy_(b.repeat_interleave(parts))
