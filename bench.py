@@ -10,7 +10,7 @@
     python bench.py --compare pimodra
     python bench.py --compare nukelix
     python bench.py --compare lurisun
-                    (Bolonex beside Gemma 2, or Petanex beside Bolonex, at equal layer sizes: prefill and decode throughput
+                    (Bolonex beside Gemma 2, Petanex beside Bolonex, and so on, at equal layer sizes: prefill and decode throughput
                     and, per operation, the time of one step against the time its bytes, or its multiply-adds, take at the
                     measured rates; one JSON line)
 
@@ -847,8 +847,7 @@ def lurisun_op_bytes(z: dict, T: int, n_reqs: int, keys: int) -> dict:
                             n_att * 4 * H * d * pairs_c + n_lat * 4 * lh * D * pairs_w),
         "decay_memory": n_lig * (T * mh * (2 * md + mv) * (4 if single else 2) + T * mh * mv * 4 + 2 * n_reqs * mh * md * mv * 4),
         "head_norm_gate": n_lig * T * mh * mv * 10,
-        "latent_append": n_lat * T * (rank * 4 + 4 * D),
-        "cols_rmsnorm": n_lat * T * z["q_rank"] * 6,
+        "latent_norms_append": n_lat * T * (rank * 4 + 4 * D + z["q_rank"] * 6),
         "head_linear": (n_lat * T * lh * (4 * d + 2 * D + 2 * D + 2 * d), n_lat * 4 * T * lh * D * d),
         "element_gate": n_lat * T * lh * d * 8,
         "add_rmsnorm": (L if single else 2 * L) * T * W * 14,
