@@ -821,7 +821,7 @@ def lurisun_config(z: dict) -> dict:
     layers = [{"type": kinds[i % 4], "mixer": (lat, lig, att, lig)[i % 4], "mlp": {"kind": "dense", "ff": z["ff"]}}
               for i in range(COMPARE_LAYERS)]
     return {"architecture": "Lurisun", "width": z["width"], "vocab": COMPARE_VOCAB, "norm": {"eps": 1e-6}, "logit_scale": 1.0,
-            "canon": {"taps": 4}, "embedding": {"bigram": {"mul_prev": 31, "mul_cur": 17, "buckets": COMPARE_VOCAB}}, "layers": layers}
+            "canon": {"taps": 4}, "embedding": {"bigram": {"mul_prev": 1009, "mul_cur": 1, "buckets": COMPARE_VOCAB}}, "layers": layers}
 
 
 def lurisun_op_bytes(z: dict, T: int, n_reqs: int, keys: int) -> dict:

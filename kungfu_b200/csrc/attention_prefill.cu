@@ -151,32 +151,32 @@ attn_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
       }
     }
     if constexpr (!SIG) {
-    float corr[2];
+      float corr[2];
 #pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      m_new[r] = fmaxf(m_new[r], __shfl_xor_sync(0xffffffffu, m_new[r], 1));
-      m_new[r] = fmaxf(m_new[r], __shfl_xor_sync(0xffffffffu, m_new[r], 2));
-      corr[r] = (m_new[r] == -INFINITY) ? 1.f : exp2f(m_run[r] - m_new[r]);
-      m_run[r] = m_new[r];
-    }
-    float l_add[2] = {0.f, 0.f};
-#pragma unroll
-    for (int n = 0; n < NT_S; ++n) {
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int r = e >> 1;
-        const float p = (m_new[r] == -INFINITY) ? 0.f : exp2f(s_acc[n][e] - m_new[r]);
-        s_acc[n][e] = p;
-        l_add[r] += p;
+      for (int r = 0; r < 2; ++r) {
+        m_new[r] = fmaxf(m_new[r], __shfl_xor_sync(0xffffffffu, m_new[r], 1));
+        m_new[r] = fmaxf(m_new[r], __shfl_xor_sync(0xffffffffu, m_new[r], 2));
+        corr[r] = (m_new[r] == -INFINITY) ? 1.f : exp2f(m_run[r] - m_new[r]);
+        m_run[r] = m_new[r];
       }
-    }
+      float l_add[2] = {0.f, 0.f};
 #pragma unroll
-    for (int r = 0; r < 2; ++r) l_run[r] = l_run[r] * corr[r] + l_add[r];     // quad partial sums; merged at the end
+      for (int n = 0; n < NT_S; ++n) {
 #pragma unroll
-    for (int n = 0; n < NT_O; ++n) {
-      o_acc[n][0] *= corr[0]; o_acc[n][1] *= corr[0];
-      o_acc[n][2] *= corr[1]; o_acc[n][3] *= corr[1];
-    }
+        for (int e = 0; e < 4; ++e) {
+          const int r = e >> 1;
+          const float p = (m_new[r] == -INFINITY) ? 0.f : exp2f(s_acc[n][e] - m_new[r]);
+          s_acc[n][e] = p;
+          l_add[r] += p;
+        }
+      }
+#pragma unroll
+      for (int r = 0; r < 2; ++r) l_run[r] = l_run[r] * corr[r] + l_add[r];     // quad partial sums; merged at the end
+#pragma unroll
+      for (int n = 0; n < NT_O; ++n) {
+        o_acc[n][0] *= corr[0]; o_acc[n][1] *= corr[0];
+        o_acc[n][2] *= corr[1]; o_acc[n][3] *= corr[1];
+      }
     }
     // ---- O += P V -----------------------------------------------------------------------------------------------
 #pragma unroll

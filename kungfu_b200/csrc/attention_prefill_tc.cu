@@ -475,35 +475,35 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
           pk[(c >> 1) + 1] = *reinterpret_cast<const uint32_t*>(&b1);
         }
       } else {
-      float mt[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+        float mt[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
-      for (int c = 0; c < BKV; c += 8) {
-        mt[0] = max3(mt[0], sv[c], sv[c + 1]); mt[1] = max3(mt[1], sv[c + 2], sv[c + 3]);
-        mt[2] = max3(mt[2], sv[c + 4], sv[c + 5]); mt[3] = max3(mt[3], sv[c + 6], sv[c + 7]);
-      }
-      const float m_tile = fmaxf(fmaxf(mt[0], mt[1]), fmaxf(mt[2], mt[3]));
-      // the maximum O is scaled to after tile i - 1, from the other group; this tile's goes back the same way
-      if (i > 0) ok = ok && mbar_wait(&m_done[grp ^ 1], ((i - 1) >> 1) & 1);
-      const float m_used = i > 0 ? s_max[r] : -INFINITY;
-      raise = m_tile > m_used + RESCALE_STEP;   // also true for the first finite maximum
-      const float m_new = raise ? m_tile : m_used;
-      s_max[r] = m_new;
-      mbar_arrive(&m_done[grp]);
-      corr = raise ? ex2_fast(m_used - m_new) : 1.f;   // for O; exp2(-inf) = 0 when nothing was accumulated yet
-      const float m_sub = (m_new == -INFINITY) ? 0.f : m_new;      // a row that has seen nothing yet: exp2(-inf - 0) = 0
-      const float l_corr = (m_mine == m_new) ? 1.f : ex2_fast(m_mine - m_new);   // this group's sum follows the maximum
-      float2 la[4] = {{0.f, 0.f}, {0.f, 0.f}, {0.f, 0.f}, {0.f, 0.f}};   // four chains of packed sums; the order is fixed
-      const float2 neg_m = make_float2(-m_sub, -m_sub);
+        for (int c = 0; c < BKV; c += 8) {
+          mt[0] = max3(mt[0], sv[c], sv[c + 1]); mt[1] = max3(mt[1], sv[c + 2], sv[c + 3]);
+          mt[2] = max3(mt[2], sv[c + 4], sv[c + 5]); mt[3] = max3(mt[3], sv[c + 6], sv[c + 7]);
+        }
+        const float m_tile = fmaxf(fmaxf(mt[0], mt[1]), fmaxf(mt[2], mt[3]));
+        // the maximum O is scaled to after tile i - 1, from the other group; this tile's goes back the same way
+        if (i > 0) ok = ok && mbar_wait(&m_done[grp ^ 1], ((i - 1) >> 1) & 1);
+        const float m_used = i > 0 ? s_max[r] : -INFINITY;
+        raise = m_tile > m_used + RESCALE_STEP;   // also true for the first finite maximum
+        const float m_new = raise ? m_tile : m_used;
+        s_max[r] = m_new;
+        mbar_arrive(&m_done[grp]);
+        corr = raise ? ex2_fast(m_used - m_new) : 1.f;   // for O; exp2(-inf) = 0 when nothing was accumulated yet
+        const float m_sub = (m_new == -INFINITY) ? 0.f : m_new;      // a row that has seen nothing yet: exp2(-inf - 0) = 0
+        const float l_corr = (m_mine == m_new) ? 1.f : ex2_fast(m_mine - m_new);   // this group's sum follows the maximum
+        float2 la[4] = {{0.f, 0.f}, {0.f, 0.f}, {0.f, 0.f}, {0.f, 0.f}};   // four chains of packed sums; the order is fixed
+        const float2 neg_m = make_float2(-m_sub, -m_sub);
 #pragma unroll
-      for (int c = 0; c < BKV; c += 2) {
-        const float2 x = __fadd2_rn(make_float2(sv[c], sv[c + 1]), neg_m);
-        const float2 pp = make_float2(ex2_fast(x.x), ex2_fast(x.y));
-        la[(c >> 1) & 3] = __fadd2_rn(la[(c >> 1) & 3], pp);
-        const __nv_bfloat162 b = __floats2bfloat162_rn(pp.x, pp.y);
-        pk[c >> 1] = *reinterpret_cast<const uint32_t*>(&b);
-      }
-      l_sum = l_sum * l_corr + (((la[0].x + la[0].y) + (la[1].x + la[1].y)) + ((la[2].x + la[2].y) + (la[3].x + la[3].y)));
-      m_mine = m_new;
+        for (int c = 0; c < BKV; c += 2) {
+          const float2 x = __fadd2_rn(make_float2(sv[c], sv[c + 1]), neg_m);
+          const float2 pp = make_float2(ex2_fast(x.x), ex2_fast(x.y));
+          la[(c >> 1) & 3] = __fadd2_rn(la[(c >> 1) & 3], pp);
+          const __nv_bfloat162 b = __floats2bfloat162_rn(pp.x, pp.y);
+          pk[c >> 1] = *reinterpret_cast<const uint32_t*>(&b);
+        }
+        l_sum = l_sum * l_corr + (((la[0].x + la[0].y) + (la[1].x + la[1].y)) + ((la[2].x + la[2].y) + (la[3].x + la[3].y)));
+        m_mine = m_new;
       }
       if (i > 0) {                                          // P V of the previous tile must be done: O is at rest, P is free
         ok = ok && mbar_wait(&pv_done[(i - 1) & 1], ((i - 1) >> 1) & 1);
@@ -536,14 +536,14 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_co
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     float m_used = 0.f;
     if constexpr (!SIG) {
-    // the row's sum is the two groups' sums, both brought to the last maximum; every softmax thread reaches this
-    asm volatile("bar.sync 2, 256;" ::: "memory");          // every tile's maximum has been published
-    m_used = n_tiles > 0 ? s_max[r] : -INFINITY;
-    l_sum = (m_mine == m_used) ? l_sum : l_sum * ex2_fast(m_mine - m_used);
-    asm volatile("bar.sync 2, 256;" ::: "memory");          // ... and read by both threads of the row
-    s_max[half * BMQ + r] = l_sum;
-    asm volatile("bar.sync 2, 256;" ::: "memory");
-    l_sum = s_max[r] + s_max[BMQ + r];
+      // the row's sum is the two groups' sums, both brought to the last maximum; every softmax thread reaches this
+      asm volatile("bar.sync 2, 256;" ::: "memory");          // every tile's maximum has been published
+      m_used = n_tiles > 0 ? s_max[r] : -INFINITY;
+      l_sum = (m_mine == m_used) ? l_sum : l_sum * ex2_fast(m_mine - m_used);
+      asm volatile("bar.sync 2, 256;" ::: "memory");          // ... and read by both threads of the row
+      s_max[half * BMQ + r] = l_sum;
+      asm volatile("bar.sync 2, 256;" ::: "memory");
+      l_sum = s_max[r] + s_max[BMQ + r];
     } else {
       l_sum = part == 0 ? 1.f : 0.f;
     }
