@@ -3,6 +3,8 @@
 //   o_t = S_t^T q_t
 // q, k, v are column ranges of rows laid out head by head: either 32-bit projection results, to which an activation is
 // applied as they are read (act 1: silu), or bfloat16 rows that have been through it.  Results are 32-bit [rows, H dv].
+// q and k may be turned as they are read (32-bit rows): pairs (i, i + rot/2) of every head's first `rot` elements by the
+// step's cos/sin table, k then multiplied by `kscale`; decay_rotate_kernel does the same ahead of the tensor cores.
 // `powers` [H, n_powers] holds a_h^0, a_h^1, ... (made in 64-bit on the host): a decay is never the result of a device-side
 // power, and ratios a^i / a^j never appear, so any decay in [0, 1] is exact.
 //
@@ -36,7 +38,20 @@ struct DecayArgs {
   int H, d, dv, n_reqs;
   const int* row_start; const int* n_rows; const int* slot;
   int writes;
+  const float* cos; const float* sin; int rot;       // 0: nothing is turned
+  float kscale;
 };
+
+// Element i of a head of q or k at row t: activated, then turned.
+template <typename T>
+__device__ __forceinline__ float dm_turned(const DecayArgs& a, const T* p, const float* cos, const float* sin, int t, int i) {
+  const float x = dm_act(kf_load(p, i), a.act);
+  if (i >= a.rot) return x;
+  const int half = a.rot >> 1, e = i < half ? i : i - half;
+  const float y = dm_act(kf_load(p, i < half ? i + half : e), a.act);
+  const float c = cos[(size_t)t * half + e], s = sin[(size_t)t * half + e];
+  return i < half ? fmaf(x, c, -y * s) : fmaf(x, c, y * s);
+}
 
 // ---- one row per request -------------------------------------------------------------------------------------------
 
@@ -69,9 +84,11 @@ __global__ void __launch_bounds__(DD_THREADS) decay_decode_kernel(DecayArgs p) {
   const T* q = kf_produced((const T*)p.q) + (size_t)t * p.ldq + h * p.d;
   const T* k = kf_produced((const T*)p.k) + (size_t)t * p.ldk + h * p.d;
   const T* v = kf_produced((const T*)p.v) + (size_t)t * p.ldv + h * p.dv;
+  const float* cos = kf_produced(p.cos);
+  const float* sin = kf_produced(p.sin);
   for (int i = tid; i < p.d; i += DD_THREADS) {
-    qs[i] = dm_act(kf_load(q, i), p.act);
-    ks[i] = dm_act(kf_load(k, i), p.act);
+    qs[i] = dm_turned(p, q, cos, sin, t, i);
+    ks[i] = dm_turned(p, k, cos, sin, t, i) * p.kscale;
   }
   if (tid < DD_COLS && tile * DD_COLS + tid < p.dv) vs[tid] = dm_act(kf_load(v, tile * DD_COLS + tid), p.act);
   __syncthreads();
@@ -143,8 +160,8 @@ __global__ void __launch_bounds__(LANES * DW_COLS) decay_walk_kernel(DecayArgs p
     for (int i = tid; i < rows * DP; i += THREADS) {
       const int t = i / DP, e = i - t * DP;
       const size_t row = (size_t)(row0 + c0 + t);
-      qs[t][e] = e < p.d ? dm_act(kf_load(qg, row * p.ldq + e), p.act) : 0.f;
-      ks[t][e] = e < p.d ? dm_act(kf_load(kg, row * p.ldk + e), p.act) : 0.f;
+      qs[t][e] = e < p.d ? dm_turned(p, qg + row * p.ldq, p.cos, p.sin, (int)row, e) : 0.f;
+      ks[t][e] = e < p.d ? dm_turned(p, kg + row * p.ldk, p.cos, p.sin, (int)row, e) * p.kscale : 0.f;
     }
     for (int i = tid; i < rows * DW_COLS; i += THREADS) {
       const int t = i / DW_COLS, c = cb * DW_COLS + (i - t * DW_COLS);
@@ -471,6 +488,52 @@ decay_chunk_starts_kernel(DecayArgs p, int chunk_rows, float* __restrict__ chunk
   }
 }
 
+// From 32-bit projection rows to the bfloat16 rows [q | k | v] the tensor-core kernel reads: q and k turned, k scaled.
+// One thread per four neighbouring elements (V = 4: rot and d multiples of eight, dv and the columns of four), or per element.
+template <int V>
+__global__ void __launch_bounds__(256)
+decay_rotate_kernel(const float* __restrict__ in, int ld, int q0, int k0, int v0, const float* __restrict__ cos,
+                    const float* __restrict__ sin, int rot, float kscale, int H, int d, int dv, __nv_bfloat16* __restrict__ out,
+                    int T) {
+  kf_pdl_trigger();
+  kf_pdl_wait();
+  const int nq = H * d, width = 2 * nq + H * dv, per = width / V, half = rot >> 1;
+  const long item = (long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (item >= (long)T * per) return;
+  const int t = (int)(item / per), c = (int)(item - (long)t * per) * V;
+  const float* row = in + (size_t)t * ld;
+  float x[V];
+  auto read = [&](const float* p, float* o) {
+    if constexpr (V == 4) { const float4 f = *reinterpret_cast<const float4*>(p); o[0] = f.x, o[1] = f.y, o[2] = f.z, o[3] = f.w; }
+    else o[0] = *p;
+  };
+  if (c >= 2 * nq) {
+    read(row + v0 + c - 2 * nq, x);
+  } else {
+    const bool key = c >= nq;
+    const int cc = key ? c - nq : c, i = cc % d;
+    const float* src = row + (key ? k0 : q0) + cc;
+    read(src, x);
+    if (i < rot) {
+      const bool low = i < half;
+      const int e = low ? i : i - half;
+      float y[V], cs[V], sn[V];
+      read(src + (low ? half : -half), y);
+      read(cos + (size_t)t * half + e, cs);
+      read(sin + (size_t)t * half + e, sn);
+#pragma unroll
+      for (int u = 0; u < V; ++u) x[u] = fmaf(x[u], cs[u], low ? -y[u] * sn[u] : y[u] * sn[u]);
+    }
+    if (key) {
+#pragma unroll
+      for (int u = 0; u < V; ++u) x[u] *= kscale;
+    }
+  }
+  __nv_bfloat16* o = out + (size_t)t * width + c;
+  if constexpr (V == 4) *reinterpret_cast<uint2*>(o) = make_uint2(kf_mma::pack_bf16(x[0], x[1]), kf_mma::pack_bf16(x[2], x[3]));
+  else *o = __float2bfloat16_rn(x[0]);
+}
+
 template <int D, int VT, int WARPS>
 int launch_chunks(const DecayArgs& p, int mode, int chunk_rows, int n_numbers, float* chunk_state, cudaStream_t stream) {
   const size_t smem = (size_t)(4 * DC_ROWS * D + 2 * DC_ROWS * VT + 2 * D * VT) * 2 + (DC_ROWS + 1) * sizeof(float);
@@ -504,20 +567,36 @@ KF_API int kf_decay_chunk_supported(int d, int dv, int ld) {
 // Blocks per (request, head) of that kernel.
 KF_API int kf_decay_chunk_tiles(int d, int dv) { return kf_ceil_div(dv, d <= 128 ? 64 : 32); }
 
+// in [T, ld] 32-bit with q, k, v in columns q0, k0, v0; out [T, 2 H d + H dv] bfloat16.
+KF_API int kf_decay_rotate(const float* in, int ld, int q0, int k0, int v0, const float* cos, const float* sin, int rot, float kscale,
+                           int H, int d, int dv, void* out, int T, cudaStream_t stream) {
+  if (T <= 0) return KF_OK;
+  if (H < 1 || d < 1 || dv < 1 || rot < 0 || rot > d || (rot & 1) || (rot && (!cos || !sin))) return KF_ERR_SIZE;
+  const bool by4 = rot % 8 == 0 && d % 8 == 0 && dv % 4 == 0 && ((ld | q0 | k0 | v0) & 3) == 0 &&
+                   (((uintptr_t)in | (uintptr_t)out | (uintptr_t)cos | (uintptr_t)sin) & 15) == 0;
+  const long n = (long)T * (2 * H * d + H * dv) / (by4 ? 4 : 1);
+  const dim3 grid((unsigned)((n + 255) / 256));
+  if (by4) kf_launch(decay_rotate_kernel<4>, grid, dim3(256), 0, stream, in, ld, q0, k0, v0, cos, sin, rot, kscale, H, d, dv, (__nv_bfloat16*)out, T);
+  else kf_launch(decay_rotate_kernel<1>, grid, dim3(256), 0, stream, in, ld, q0, k0, v0, cos, sin, rot, kscale, H, d, dv, (__nv_bfloat16*)out, T);
+  KF_CHECK_LAUNCH();
+  return KF_OK;
+}
+
 // rows: the base of the matrix that holds q, k and v in columns q0, k0, v0 (`ld` columns); dtype: its element type.
 // chunk_rows > 0 (a multiple of 64, below n_powers): chunks side by side; chunk_state then holds n_numbers * H * d * dv
 // floats, n_numbers at least the number of chunks of the step.  single: no request has more than one row.
 KF_API int kf_decay_memory(const void* rows, int dtype, int ld, int q0, int k0, int v0, int act, const float* powers,
                            int n_powers, float* state, float* out, int H, int d, int dv, int n_reqs, const int* row_start,
                            const int* n_rows, const int* slot, int writes, int single, int chunk_rows, int n_numbers,
-                           float* chunk_state, cudaStream_t stream) {
+                           float* chunk_state, const float* cos, const float* sin, int rot, float kscale, cudaStream_t stream) {
   if (n_reqs <= 0) return KF_OK;
+  if (rot < 0 || rot > d || (rot & 1) || (rot && (!cos || !sin))) return KF_ERR_SIZE;
   if (d < 1 || d > 256 || dv < 1 || H < 1 || n_powers < DC_ROWS + 1) return KF_ERR_SIZE;
   if (dtype != KF_F32 && dtype != KF_BF16) return KF_ERR_DTYPE;
   const size_t es = dtype == KF_F32 ? 4 : 2;
   const char* base = (const char*)rows;
   DecayArgs p{base + q0 * es, base + k0 * es, base + v0 * es, ld, ld, ld, act, powers, n_powers, state, out, H, d, dv, n_reqs,
-              row_start, n_rows, slot, writes};
+              row_start, n_rows, slot, writes, cos, sin, rot, kscale};
   if (single && dv % 4 == 0 && (((uintptr_t)state | (uintptr_t)out) & 15) == 0) {
     const dim3 grid((unsigned)((long)n_reqs * H * kf_ceil_div(dv, DD_COLS)));
 #define KF_GO(NR)                                                                                               \
@@ -530,7 +609,7 @@ KF_API int kf_decay_memory(const void* rows, int dtype, int ld, int q0, int k0, 
     KF_CHECK_LAUNCH();
     return KF_OK;
   }
-  if (dtype == KF_BF16 && act == 0 && kf_decay_chunk_supported(d, dv, ld) && ((q0 | k0 | v0) & 7) == 0 &&
+  if (dtype == KF_BF16 && act == 0 && rot == 0 && kscale == 1.f && kf_decay_chunk_supported(d, dv, ld) && ((q0 | k0 | v0) & 7) == 0 &&
       (((uintptr_t)rows | (uintptr_t)state | (uintptr_t)chunk_state) & 15) == 0) {
     if (chunk_rows <= 0) return chunk_pass(p, DC_WHOLE, 1 << 30, n_reqs, state, stream);
     if (chunk_rows % DC_ROWS || chunk_rows >= n_powers || !chunk_state || n_numbers < 1) return KF_ERR_SIZE;

@@ -273,7 +273,7 @@ KF_API int kf_delta_rule(const float* qkv, int ld_qkv, int q0, int k0, int v0, c
 }
 
 // out[t, h*dv + i] = o[t, h*dv + i] / sqrt(mean_i(o[t, h, :]^2) + eps) * w[i] * act(gate[t, gate0 + h*dv + i]),
-// act: 0 = silu, 1 = sigmoid.  One warp per (row, head).
+// act: 0 = silu, 1 = sigmoid; w null: no weight.  One warp per (row, head).
 template <typename TW, typename TO>
 __global__ void head_norm_gate_kernel(const float* __restrict__ o, const TW* __restrict__ w, float eps,
                                       const float* __restrict__ gate, int ld_gate, int gate0, int act,
@@ -293,7 +293,7 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, const TW* __r
   for (int i = lane; i < dv; i += 32) {
     const float z = g[i];
     const float s = 1.f / (1.f + expf(-z));
-    kf_store(out, (size_t)t * ldo + ocol0 + h * dv + i, src[i] * inv * kf_load(w, h * w_stride + i) * (act == 0 ? z * s : s) * scale);
+    kf_store(out, (size_t)t * ldo + ocol0 + h * dv + i, src[i] * inv * (w ? kf_load(w, h * w_stride + i) : 1.f) * (act == 0 ? z * s : s) * scale);
   }
 }
 
@@ -310,7 +310,7 @@ head_norm_gate_block_kernel(const float* o, const TW* __restrict__ w, float eps,
 #pragma unroll
   for (int k = 0; k < NPT; ++k) {
     const int i = threadIdx.x + k * blockDim.x;
-    wv[k] = i < dv ? kf_load(w, h * w_stride + i) : 0.f;
+    wv[k] = i < dv ? (w ? kf_load(w, h * w_stride + i) : 1.f) : 0.f;
   }
   kf_pdl_wait();
   o = kf_produced(o), gate = kf_produced(gate);

@@ -1,11 +1,11 @@
 // Embedding gather, rotary tables, gated activation, residual add.
 #include "common.cuh"
 
-// x[t, :] = table[token[t], :] * scale.  A token id outside [0, V) writes zeros and sets *bad.
+// x[t, :] = table[token[t], :] * scale, `copies` times over (x [rows, copies, H]).  A token id outside [0, V) writes zeros and sets *bad.
 // Reference: gather then scale, crates/kf-layers/src/basic.rs:35-36.
 template <typename TW>
 __global__ void embed_kernel(const int* __restrict__ tokens, const TW* __restrict__ table, float scale,
-                             float* __restrict__ out, int H, int V, int* __restrict__ bad) {
+                             float* __restrict__ out, int H, int V, int copies, int* __restrict__ bad) {
   kf_pdl_trigger();
   kf_pdl_wait();
   const int t = blockIdx.x;
@@ -13,18 +13,22 @@ __global__ void embed_kernel(const int* __restrict__ tokens, const TW* __restric
   const bool ok = tok >= 0 && tok < V;
   if (!ok && threadIdx.x == 0 && bad) atomicExch(bad, 1);
   const TW* row = table + (size_t)(ok ? tok : 0) * H;
-  float* o = out + (size_t)t * H;
-  for (int i = threadIdx.x; i < H; i += blockDim.x) o[i] = ok ? kf_load(row, i) * scale : 0.f;
+  float* o = out + (size_t)t * copies * H;
+  for (int i = threadIdx.x; i < H; i += blockDim.x) {
+    const float v = ok ? kf_load(row, i) * scale : 0.f;
+    for (int c = 0; c < copies; ++c) o[(size_t)c * H + i] = v;
+  }
 }
 
 KF_API int kf_embed(const int* tokens, const void* table, int table_dtype, float scale, float* out,
-                    int T, int H, int V, int* bad_flag, cudaStream_t stream) {
+                    int T, int H, int V, int copies, int* bad_flag, cudaStream_t stream) {
   if (T <= 0) return KF_OK;
+  if (copies < 1) return KF_ERR_SIZE;
   const int threads = H >= 1024 ? 256 : 128;
   if (table_dtype == KF_F32)
-    kf_launch(embed_kernel<float>, dim3(T), dim3(threads), 0, stream, tokens, (const float*)table, scale, out, H, V, bad_flag);
+    kf_launch(embed_kernel<float>, dim3(T), dim3(threads), 0, stream, tokens, (const float*)table, scale, out, H, V, copies, bad_flag);
   else if (table_dtype == KF_BF16)
-    kf_launch(embed_kernel<__nv_bfloat16>, dim3(T), dim3(threads), 0, stream, tokens, (const __nv_bfloat16*)table, scale, out, H, V, bad_flag);
+    kf_launch(embed_kernel<__nv_bfloat16>, dim3(T), dim3(threads), 0, stream, tokens, (const __nv_bfloat16*)table, scale, out, H, V, copies, bad_flag);
   else
     return KF_ERR_DTYPE;
   KF_CHECK_LAUNCH();

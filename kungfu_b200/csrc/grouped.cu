@@ -16,7 +16,8 @@
 //   groups of neighbouring experts ranked by the sum of their two largest choice scores (or, `group_best` = 1, by their
 //   largest), the best `keep` groups stay eligible, the `top` largest eligible choice scores win (lower index first
 //   among equals); weights = the winners' uncorrected scores, divided by their sum + 1e-20 when `normalize`, times
-//   `scale`.  One warp per token, everything 32-bit.
+//   `scale`.  `softmax` 2: the correction is part of the logit, the choice is made on the logits and the weights are the
+//   softmax over the chosen logits alone, times `scale`.  One warp per token, everything 32-bit.
 // kf_moe_plan: counts the pairs of every expert, lays the pairs out expert by expert (sorted_pair, inverse), and lists
 //   the row tiles of every expert.  One block; the order inside an expert is whatever the atomics give, which no
 //   result depends on (a pair's output row is computed from its own row alone).
@@ -316,14 +317,20 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict_
   float* gscore = choice + E;
   const float NEG = -INFINITY;
   float zmax = NEG, zsum = 0.f;
-  if (softmax) {
+  if (softmax == 1) {
     for (int e = lane; e < E; e += 32) zmax = fmaxf(zmax, logits[(size_t)t * E + e]);
     zmax = kf_warp_max(zmax);
     for (int e = lane; e < E; e += 32) zsum += expf(logits[(size_t)t * E + e] - zmax);
     zsum = kf_warp_sum(zsum);
   }
   for (int e = lane; e < E; e += 32) {
-    const float z = logits[(size_t)t * E + e];
+    float z = logits[(size_t)t * E + e];
+    if (softmax == 2) {                                // the biased logit is the score and the choice
+      if (correction) z += kf_load(correction, e);
+      score[e] = z;
+      choice[e] = (z == z && z != INFINITY) ? z : NEG;
+      continue;
+    }
     const float s = softmax ? expf(z - zmax) / zsum : 1.f / (1.f + expf(-z));
     score[e] = s;
     // sigmoid scores without a correction and without groups rank as their logits do, and the logits do not run into
@@ -383,6 +390,15 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict_
     }
     __syncwarp();
     sum += score[arg];
+  }
+  if (softmax == 2) {
+    const float most = score[ids[(size_t)t * top]];    // the first choice
+    float all = 0.f;
+    for (int r = lane; r < top; r += 32) all += expf(score[ids[(size_t)t * top + r]] - most);
+    all = kf_warp_sum(all);
+    for (int r = lane; r < top; r += 32)
+      weights[(size_t)t * top + r] = expf(score[ids[(size_t)t * top + r]] - most) / all * scale;
+    return;
   }
   for (int r = lane; r < top; r += 32) {
     const int e = ids[(size_t)t * top + r];

@@ -257,10 +257,12 @@ def attention_head_size(n: int) -> int:
 
 @_dispatch("embed")
 def embed(tokens, table, scale: float, out) -> None:
-    """out[t, :] = table[tokens[t], :] * scale (32-bit out).  Token ids are validated by the caller on the host."""
+    """out[t, :] = table[tokens[t], :] * scale (32-bit out); out [T, n, width]: n copies of every row.  Token ids are
+    validated by the caller on the host."""
     T, (V, H) = out.shape[0], table.shape
-    _check(library().kf_embed(_p(tokens), _p(table), _dt(table), _f(scale), _p(out), T, H, V, ctypes.c_void_p(0), _stream()),
-           "embed")
+    copies = out.shape[1] if out.dim() == 3 else 1
+    _check(library().kf_embed(_p(tokens), _p(table), _dt(table), _f(scale), _p(out), T, H, V, int(copies), ctypes.c_void_p(0),
+                              _stream()), "embed")
 
 
 @_dispatch("rmsnorm")
@@ -654,16 +656,20 @@ def short_conv_commit(proj, col0: int, in_bias, n_channels: int, taps: int, stat
 @_dispatch("qkv_prepare")
 def qkv_prepare(proj, col0: int, in_bias, conv_w, conv_state, q_norm, k_norm, eps: float, cos, sin, rot: int,
                 interleaved: bool, n_heads: int, n_kv_heads: int, key_dim: int, value_dim: int, ctx, cache, q_out,
-                commit_inline: bool = False) -> bool:
+                commit_inline: bool = False, parts: int = 1, temperature: tuple | None = None) -> bool:
     """From the 32-bit q|k|v projection to the attention's operands: optional bias, short convolution (reading
     `conv_state`), per-head RMS norm of q and k, rotation (interleaved pairs or halves), q into `q_out`
-    [T, n_heads * D] and k, v into the pages of `cache`, D = the pages' head size, tails zero.
+    [T, n_heads * parts * D] and k, v into the pages of `cache`, D = the pages' head size, tails zero.
+    `parts` > 1: a head of q and of k is that many vectors of key_dim, each with a rotation of its own; the parts of k stand
+    side by side in one stored key, part m of q becomes query head h * parts + m, zero outside its part's place.
+    `temperature` (coef, every): q times 1 + coef ln(floor((position + 1) / every) + 1), after the rotation.
     `commit_inline` (only for steps in which no request has more than one row): the kernel also moves the convolution's
     state on, when its sizes allow.  Returns whether it did; if not, `short_conv_commit` has to run afterwards."""
     T = q_out.shape[0]
     D = cache.pages.shape[-1]
-    if q_out.shape[1] != n_heads * D:
-        raise KernelError(f"qkv_prepare: q rows of {q_out.shape[1]} elements for {n_heads} heads of {D}")
+    if q_out.shape[1] != n_heads * parts * D:
+        raise KernelError(f"qkv_prepare: q rows of {q_out.shape[1]} elements for {n_heads} heads of {parts} x {D}")
+    coef, every = temperature if temperature is not None else (0.0, 1)
     table = ctx.block_tables[cache.group]
     taps = conv_w.shape[1] if conv_w is not None else 1
     wdt = _dt(conv_w) if conv_w is not None else _dt(q_out)
@@ -671,12 +677,13 @@ def qkv_prepare(proj, col0: int, in_bias, conv_w, conv_state, q_norm, k_norm, ep
         if w is not None and _dt(w) != wdt:
             raise KernelError("qkv_prepare: bias, convolution and norm weights must share one element type")
     inline = bool(commit_inline and conv_w is not None and taps > 1 and conv_state is not None and
-                  library().kf_qkv_prepare_commits_inline(proj.shape[1], int(col0), int(rot), int(interleaved), key_dim, value_dim, D))
+                  library().kf_qkv_prepare_commits_inline(proj.shape[1], int(col0), int(rot), int(interleaved), key_dim, value_dim, D,
+                                                          int(parts), _f(coef)))
     _check(library().kf_qkv_prepare(_p(proj), proj.shape[1], int(col0), _p(in_bias), _p(conv_w), taps, _p(conv_state),
                                     _p(q_norm), _p(k_norm), wdt, _f(eps), _p(cos), _p(sin), int(rot), int(interleaved),
-                                    n_heads, n_kv_heads, key_dim, value_dim, D, _p(ctx.positions), _p(ctx.row_req),
-                                    _p(ctx.req_row_start), _p(ctx.req_state_slot), _p(table), table.shape[1],
-                                    cache.page_size, _p(cache.pages), _dt(cache.pages), _p(q_out), _dt(q_out),
+                                    n_heads, n_kv_heads, key_dim, value_dim, D, int(parts), _f(coef), int(every),
+                                    _p(ctx.positions), _p(ctx.row_req), _p(ctx.req_row_start), _p(ctx.req_state_slot), _p(table),
+                                    table.shape[1], cache.page_size, _p(cache.pages), _dt(cache.pages), _p(q_out), _dt(q_out),
                                     int(cache.writes), T, int(inline), _stream()), "qkv_prepare")
     return inline
 
@@ -697,6 +704,19 @@ SCAN_CHUNK_ROWS = 256
 SCAN_CHUNKED_FROM = 1024     # rows of a step from which the chunks are walked side by side ...
 SCAN_CHUNKED_BLOCKS = 160    # ... if the plain walk would have at most this many blocks (about one per SM); with two per SM
                              # it is already the faster one (736 against 827 us at 128 heads x 64 x 128)
+
+
+@_dispatch("diff_combine")
+def diff_combine(o, lam: float, factor: float, eps: float, proj, gate_col0: int, n_heads: int, value_dim: int, head_dim: int, out,
+                 ctx) -> None:
+    """out[t, h, :] = d / sqrt(mean(d^2) + eps) * factor * sigmoid(proj[t, gate_col0 + h]), d = o[t, 2h, :] - lam * o[t, 2h + 1, :]
+    over the first value_dim of head_dim elements; proj None: no gate."""
+    T = out.shape[0]
+    if o.shape[1] != 2 * n_heads * head_dim or out.shape[1] != n_heads * value_dim or o.dtype != out.dtype:
+        raise KernelError(f"diff_combine: o{tuple(o.shape)} {o.dtype} and out{tuple(out.shape)} {out.dtype} do not fit {n_heads} heads")
+    _check(library().kf_diff_combine(_p(o), _f(lam), _f(factor), _f(eps), _p(proj), proj.shape[1] if proj is not None else 0,
+                                     int(gate_col0), n_heads, value_dim, head_dim, _p(out), _dt(out), _p(ctx.row_req), T,
+                                     _stream()), "diff_combine")
 
 
 @_dispatch("ssm_scan")
@@ -743,6 +763,32 @@ def add2_rmsnorm(a, b, x, *, next_weight=None, next_eps: float = 0.0, next_plus_
     _check(library().kf_add2_rmsnorm(_p(a), _p(b), _p(x), _p(next_weight), _dt(next_weight) if next_weight is not None else F32,
                                      _f(next_eps), int(next_plus_one), _p(next_out),
                                      _dt(next_out) if next_out is not None else F32, T, H, _stream()), "add2_rmsnorm")
+
+
+# ---- a residual of several streams --------------------------------------------------------------------------------------
+
+MAX_STREAMS = 16
+
+
+@_dispatch("streams_norm")
+def streams_norm(x, weights, norm_weight, eps: float, out, rows=None) -> None:
+    """out[r] = rms_norm(sum_s weights[s] * x[row, s]) * norm_weight, row = rows[r] (r without rows); x [rows, n, width] and
+    `weights` [n] 32-bit."""
+    n, W = x.shape[1], x.shape[2]
+    _check(library().kf_streams_step(_p(x), None, None, None, _p(rows), _p(weights), _p(norm_weight), _dt(norm_weight), _f(eps),
+                                     _p(out), _dt(out), out.shape[0], n, W, _stream()), "streams_norm")
+
+
+@_dispatch("streams_step")
+def streams_step(x, y, mix, out_weights, *, next_weights=None, next_norm=None, next_eps: float = 0.0, next_out=None) -> None:
+    """x[r, t] <- sum_s mix[s, t] * x[r, s] + out_weights[t] * y[r], all streams at once; if next_out is given, the
+    `streams_norm` of the new streams in the same pass.  x, y, mix [n, n] and the weights 32-bit."""
+    T, n, W = x.shape
+    if tuple(mix.shape) != (n, n) or tuple(y.shape) != (T, W):
+        raise KernelError(f"streams_step: x{tuple(x.shape)} y{tuple(y.shape)} mix{tuple(mix.shape)} do not agree")
+    _check(library().kf_streams_step(_p(x), _p(y), _p(mix), _p(out_weights), None, _p(next_weights), _p(next_norm),
+                                     _dt(next_norm) if next_norm is not None else F32, _f(next_eps), _p(next_out),
+                                     _dt(next_out) if next_out is not None else F32, T, n, W, _stream()), "streams_step")
 
 
 # ---- norms in groups, the polynomial activation, attention whose heads' weights are mixed ---------------------------------
@@ -852,13 +898,13 @@ _GATE_ACT = {"silu": 0, "sigmoid": 1}
 def head_norm_gate(o, weight, eps: float, gate, gate0: int, act: str, out, heads: int, vdim: int, out_col0: int = 0,
                    scale: float = 1.0) -> None:
     """out[t, out_col0 + h * vdim + :] = o[t, h, :] / rms(o[t, h, :]) * weight * act(gate[t, gate0 + h * vdim + :]) * scale;
-    act silu or sigmoid.  `weight` holds vdim numbers (shared by the heads) or heads * vdim (one vector per head); `out` may
-    be wider than the heads (the joined input of one output product)."""
+    act silu or sigmoid.  `weight` holds vdim numbers (shared by the heads) or heads * vdim (one vector per head), or is None
+    (every weight is one); `out` may be wider than the heads (the joined input of one output product)."""
     T = out.shape[0]
-    if weight.numel() not in (vdim, heads * vdim):
+    if weight is not None and weight.numel() not in (vdim, heads * vdim):
         raise KernelError(f"head_norm_gate: {weight.numel()} weights for {heads} heads of {vdim}")
-    w_stride = vdim if (weight.numel() == heads * vdim and heads > 1) else 0
-    _check(library().kf_head_norm_gate(_p(o), _p(weight), _dt(weight), _f(eps), _p(gate), gate.shape[1], int(gate0),
+    w_stride = vdim if (weight is not None and weight.numel() == heads * vdim and heads > 1) else 0
+    _check(library().kf_head_norm_gate(_p(o), _p(weight), _dt(weight if weight is not None else out), _f(eps), _p(gate), gate.shape[1], int(gate0),
                                        _GATE_ACT[act], _p(out), _dt(out), heads, vdim, T, w_stride, out.shape[1], int(out_col0),
                                        _f(scale), _stream()), "head_norm_gate")
 
@@ -1011,16 +1057,27 @@ def decay_memory_takes_bfloat16(dim: int, vdim: int, ld: int) -> bool:
     return bool(use_tensor_cores and library().kf_decay_chunk_supported(int(dim), int(vdim), int(ld)))
 
 
+@_dispatch("decay_rotate")
+def decay_rotate(proj, q0: int, k0: int, v0: int, cos, sin, rot: int, key_scale: float, heads: int, dim: int, vdim: int, out) -> None:
+    """bfloat16 rows [q | k | v] for `decay_memory` from columns of a 32-bit projection: the first `rot` elements of every
+    head of q and k turned in pairs (i, i + rot/2), k times `key_scale`."""
+    _check(library().kf_decay_rotate(_p(proj), proj.shape[1], int(q0), int(k0), int(v0), _p(cos), _p(sin), int(rot), _f(key_scale),
+                                     heads, dim, vdim, _p(out), out.shape[0], _stream()), "decay_rotate")
+
+
 @_dispatch("decay_memory")
 def decay_memory(rows, q0: int, k0: int, v0: int, act, powers, state, out, heads: int, dim: int, vdim: int, ctx,
-                 writes: bool = True) -> None:
+                 writes: bool = True, cos=None, sin=None, rot: int = 0, key_scale: float = 1.0) -> None:
     """S <- a_h S + k v^T, o = S^T q over the rows of every request of the step, from and into `state`
     [slots, heads, dim, vdim] (32-bit); a_h = powers[h, 1] (`decay_powers`).  q, k, v are column ranges of `rows`, laid out
     head by head: 32-bit (act 'silu' is applied to them as they are read) or bfloat16 that has been through it (act
-    None).  out: 32-bit [rows, heads * vdim].  bfloat16 rows of prompt portions run on the tensor cores; a long step with
+    None).  32-bit rows may have q and k turned as they are read, k then times `key_scale` (as `decay_rotate` does for
+    bfloat16).  out: 32-bit [rows, heads * vdim].  bfloat16 rows of prompt portions run on the tensor cores; a long step with
     few heads and requests is cut into chunks that are walked side by side (three launches)."""
     T = out.shape[0]
     lib = library()
+    if rows.dtype == torch.bfloat16 and (rot or key_scale != 1.0):
+        raise KernelError("decay_memory: bfloat16 rows are turned beforehand (decay_rotate)")
     if act not in (None, "silu"):
         raise KernelError(f"decay_memory: activation {act!r} is not one of None, silu")
     single = bool(getattr(ctx, "decode_only", False))
@@ -1039,7 +1096,7 @@ def decay_memory(rows, q0: int, k0: int, v0: int, act, powers, state, out, heads
     _check(lib.kf_decay_memory(_p(rows), _dt(rows), rows.shape[1], int(q0), int(k0), int(v0), int(act == "silu"), _p(powers),
                                powers.shape[1], _p(state), _p(out), heads, dim, vdim, ctx.n_reqs, _p(ctx.req_row_start),
                                _p(ctx.req_n_rows), _p(ctx.req_state_slot), int(writes), int(single), chunk_rows, n_numbers,
-                               _p(chunk_state), _stream()), "decay_memory")
+                               _p(chunk_state), _p(cos), _p(sin), int(rot), _f(key_scale), _stream()), "decay_memory")
     if chunk_rows:
         add_launches(2)
 
@@ -1133,12 +1190,14 @@ def moe_route(logits, correction, groups: int, keep: int, top: int, scale: float
     experts); the choice is made on s + correction, among the experts of the `keep` groups (of `groups` equal groups of
     neighbours) whose two largest choice scores sum highest (group_rank 'best': whose largest is highest);
     ids [T, top] int32 = the `top` largest; weights [T, top] = s of the chosen * scale, divided by their sum + 1e-20
-    when `normalize`."""
+    when `normalize`.  score 'softmax_chosen': the correction belongs to the logits, the choice is made on them, and the
+    weights are the softmax over the chosen logits alone, times scale."""
     T, E = logits.shape
-    if score not in ("sigmoid", "softmax") or group_rank not in ("best_two", "best"):
+    modes = {"sigmoid": 0, "softmax": 1, "softmax_chosen": 2}
+    if score not in modes or group_rank not in ("best_two", "best"):
         raise KernelError(f"moe_route: score {score!r} / group_rank {group_rank!r} are not known")
     _check(library().kf_moe_route(_p(logits), _p(correction), _dt(correction) if correction is not None else F32, T, E,
-                                  int(groups), int(keep), int(top), _f(scale), int(score == "softmax"),
+                                  int(groups), int(keep), int(top), _f(scale), modes[score],
                                   int(group_rank == "best"), int(bool(normalize)), _p(ids), _p(weights), _stream()), "moe_route")
 
 

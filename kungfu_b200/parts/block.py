@@ -11,10 +11,12 @@ The residual stream and its sums stay in 32-bit.
 """
 from __future__ import annotations
 
+import torch
+
 from .. import ops
-from .base import Block, FeedForward, Mixer, Norm, StateBundle, register_block
+from .base import Block, FeedForward, Mixer, Norm, Part, StateBundle, register_block
 from .conv import InputConv
-from .norm import RmsNorm
+from .norm import RmsNorm, StreamsNorm
 
 
 class SandwichBlock(Block):
@@ -150,3 +152,47 @@ class ScaledBlock(Block):
 
 
 register_block("scaled", ScaledBlock)
+
+
+class StreamsMix(Part):
+    """How a sublayer's result y joins a residual of n streams: x_t <- sum_s mix[s, t] x_s + out[t] y, all streams at once.
+    `mix` is indexed [from, to]; both are held in 32-bit."""
+
+    def __init__(self, mix, out):
+        self.mix, self.out = mix.to(torch.float32).contiguous(), out.to(torch.float32).contiguous()
+        if mix.numel() and tuple(mix.shape) != (out.numel(), out.numel()):
+            raise ValueError(f"a mix of {tuple(mix.shape)} does not fit {out.numel()} streams")
+
+    def add_into(self, y, x, ctx, then=None, out_dtype=None):
+        """The new streams into x; returns then(x) if `then` is given (one kernel when `then` reads streams)."""
+        if isinstance(then, StreamsNorm):
+            nxt = ctx.buf("norm_out", (x.shape[0], then.width), out_dtype)
+            ops.streams_step(x, y, self.mix, self.out, next_weights=then.streams, next_norm=then.weight, next_eps=then.eps,
+                             next_out=nxt)
+            return nxt
+        ops.streams_step(x, y, self.mix, self.out)
+        return then.forward(x, ctx, out_dtype) if then is not None else None
+
+
+class StreamsBlock(Block):
+    """A pre-norm block on a residual of several streams [rows, n, width] (hyper-connections): each sublayer reads a
+    weighted sum of the streams, normed (`StreamsNorm`), and its result is mixed into all of them (`StreamsMix`).
+    `ffn` may be None.  Every update is one 32-bit kernel that also computes what the next sublayer reads."""
+    fuses_next_norm = True
+
+    def __init__(self, pre_mixer: StreamsNorm, mixer: Mixer, mix_mixer: StreamsMix, pre_ffn: StreamsNorm | None = None,
+                 ffn: FeedForward | None = None, mix_ffn: StreamsMix | None = None):
+        self.pre_mixer, self.mixer, self.mix_mixer = pre_mixer, mixer, mix_mixer
+        self.pre_ffn, self.ffn, self.mix_ffn = pre_ffn, ffn, mix_ffn
+
+    def forward(self, x, ctx, cache, normed=None, then=None):
+        act = ctx.act_dtype
+        n = normed if normed is not None else self.pre_mixer.forward(x, ctx, act)
+        y = self.mixer.forward(n, ctx, cache)
+        if self.ffn is None:
+            return x, self.mix_mixer.add_into(y, x, ctx, then=then, out_dtype=act)
+        n = self.mix_mixer.add_into(y, x, ctx, then=self.pre_ffn, out_dtype=act)
+        return x, self.mix_ffn.add_into(self.ffn.forward(n, ctx), x, ctx, then=then, out_dtype=act)
+
+
+register_block("streams", StreamsBlock)

@@ -29,6 +29,19 @@ class Embedding(Part):
         return x
 
 
+class StreamsEmbedding(Embedding):
+    """The residual starts as `streams` equal copies of the embedded row: [rows, streams, width]."""
+
+    def __init__(self, table: torch.Tensor, streams: int, scale: float = 1.0):
+        super().__init__(table, scale)
+        self.streams = int(streams)
+
+    def forward(self, ctx, cache=None) -> torch.Tensor:
+        x = ctx.buf("residual", (ctx.n_rows, self.streams, self.width), torch.float32)
+        ops.embed(ctx.tokens, self.table, self.scale, x)
+        return x
+
+
 class PairEmbedding(Embedding):
     """x = E[token] * scale + B[row]: a second table read by the token and the one before it, row =
     (previous * mul_prev + token * mul_cur) mod buckets, buckets = B's rows - 1; a sequence's first token reads B's last

@@ -28,11 +28,13 @@ class RoutedExperts(FeedForward):
         Other mixtures of the same shape: `score` 'softmax' (scores = the softmax of z over all experts), `group_rank`
         'best' (a group scores its largest member), `normalize` False (the winners keep their scores as weights, times
         `scale`), `activation` 'silu' (experts W_down [silu(g) u]), `weight_on` 'input' (y = sum of expert_e(weight_e x):
-        the weight multiplies what the expert reads, i.e. its gate and up rows before the activation, not its result)."""
+        the weight multiplies what the expert reads, i.e. its gate and up rows before the activation, not its result).
+        `score` 'softmax_chosen': the correction is a bias of the logits, z = W_r x + correction; the winners are chosen on z
+        and weighted by the softmax over their z alone."""
         if weight_on not in ("output", "input"):
             raise ValueError(f"weight_on {weight_on!r} is not one of output, input")
         self.weight_on = weight_on
-        if score not in ("sigmoid", "softmax") or group_rank not in ("best_two", "best") or activation not in ("clamped_swish", "silu"):
+        if score not in ("sigmoid", "softmax", "softmax_chosen") or group_rank not in ("best_two", "best") or activation not in ("clamped_swish", "silu"):
             raise ValueError(f"score {score!r}, group_rank {group_rank!r} or activation {activation!r} is not known")
         self.score, self.group_rank, self.normalize, self.activation = score, group_rank, bool(normalize), activation
         self.w_router, self.correction = w_router, correction

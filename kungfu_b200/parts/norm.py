@@ -101,6 +101,26 @@ class GroupRmsNorm(Norm):
 register_norm("group_rms", GroupRmsNorm)
 
 
+class StreamsNorm(Norm):
+    """What a sublayer reads of a residual of several streams x_1 .. x_n: the RMS norm of sum_s weights[s] x_s.
+    The weights are held in 32-bit; all ones give the norm of the streams' sum (an output head)."""
+
+    def __init__(self, weights: torch.Tensor, norm: RmsNorm):
+        if norm.plus_one:
+            raise ValueError("a norm over streams multiplies by its weight as it is")
+        self.streams = weights.to(torch.float32).contiguous()
+        self.weight, self.eps, self.width = norm.weight, norm.eps, norm.width
+
+    def forward(self, x, ctx, out_dtype, rows=None):
+        n = x.shape[0] if rows is None else rows.shape[0]
+        out = ctx.buf("norm_out" if rows is None else "norm_rows_out", (n, self.width), out_dtype)
+        ops.streams_norm(x, self.streams, self.weight, self.eps, out, rows)
+        return out
+
+
+register_norm("streams", StreamsNorm)
+
+
 class NoNorm(Norm):
     """The place of a norm in a block whose sublayers read the residual stream itself: the rows pass unchanged, in the
     element type the sublayer's products take (the residual's own rows when that is 32-bit)."""

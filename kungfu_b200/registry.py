@@ -67,6 +67,9 @@ def _register_builtin() -> None:
     from .config.lurisun import LurisunConfig
     from .models import lurisun
     register("Lurisun", LurisunConfig.from_dict, lurisun.build, lurisun.tensor_specs, replace=True)
+    from .config.fovosun import FovosunConfig
+    from .models import fovosun
+    register("Fovosun", FovosunConfig.from_dict, fovosun.build, fovosun.tensor_specs, replace=True)
 
 
 _register_builtin()
