@@ -24,7 +24,28 @@ class CpuOps:
         assert nh % nkv == 0 and d % 2 == 0 and d <= largest
 
     def embed(self, tokens, table, scale, out):
-        out.copy_(table.float()[tokens.long()] * torch.tensor(scale, dtype=torch.float32))
+        x = table.float()[tokens.long()] * torch.tensor(scale, dtype=torch.float32)
+        out.copy_(x[:, None, :].expand(out.shape) if out.dim() == 3 else x)
+
+    def streams_norm(self, x, weights, norm_weight, eps, out, rows=None):
+        xs = x if rows is None else x[rows.long()]
+        u = (xs * weights[None, :, None]).sum(1)
+        out.copy_((u * torch.rsqrt(u.pow(2).mean(-1, keepdim=True) + eps) * norm_weight.float()).to(out.dtype))
+
+    def streams_step(self, x, y, mix, out_weights, *, next_weights=None, next_norm=None, next_eps=0.0, next_out=None):
+        x.copy_(torch.einsum("rsw,st->rtw", x, mix) + out_weights[None, :, None] * y[:, None, :])
+        if next_out is not None:
+            self.streams_norm(x, next_weights, next_norm, next_eps, next_out)
+
+    def diff_combine(self, o, lam, factor, eps, proj, gate_col0, nh, dv, D, out, ctx):
+        T = out.shape[0]
+        a = o.float().view(T, nh, 2, D)[..., :dv]
+        y = a[:, :, 0] - lam * a[:, :, 1]
+        y = y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps) * factor
+        if proj is not None:
+            y = y * torch.sigmoid(proj[:, gate_col0:gate_col0 + nh].float())[..., None]
+        y[ctx.row_req[:T] < 0] = 0
+        out.copy_(y.reshape(T, nh * dv).to(out.dtype))
 
     def rmsnorm(self, x, weight, eps, plus_one, out, rows=None):
         xs = x if rows is None else x[rows.long()]
@@ -175,18 +196,18 @@ class CpuOps:
             state[slot, :taps - 1] = u[-(taps - 1):]
 
     def qkv_prepare(self, proj, col0, in_bias, conv_w, conv_state, q_norm, k_norm, eps, cos, sin, rot, interleaved,
-                    nh, nkv, dk, dv, ctx, cache, q_out, commit_inline=False):
+                    nh, nkv, dk, dv, ctx, cache, q_out, commit_inline=False, parts=1, temperature=None):
         T = q_out.shape[0]
         D = cache.pages.shape[-1]
-        C = (nh + nkv) * dk + nkv * dv
+        C = (nh + nkv) * parts * dk + nkv * dv
         x = torch.zeros(T, C)
         if conv_w is not None:
             self.short_conv(proj, col0, in_bias, conv_w, None, None, conv_state, x, ctx)
         else:
             x = proj[:, col0:col0 + C].float() + (in_bias.float()[None, :] if in_bias is not None else 0.0)
-        q = x[:, :nh * dk].reshape(T, nh, dk).clone()
-        k = x[:, nh * dk:(nh + nkv) * dk].reshape(T, nkv, dk).clone()
-        v = x[:, (nh + nkv) * dk:].reshape(T, nkv, dv)
+        q = x[:, :nh * parts * dk].reshape(T, nh * parts, dk).clone()
+        k = x[:, nh * parts * dk:(nh + nkv) * parts * dk].reshape(T, nkv * parts, dk).clone()
+        v = x[:, (nh + nkv) * parts * dk:].reshape(T, nkv, dv)
         for y, w in ((q, q_norm), (k, k_norm)):
             if w is not None:
                 y.copy_(y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps) * w.float())
@@ -201,11 +222,16 @@ class CpuOps:
                     a, b = y[..., :rot // 2].clone(), y[..., rot // 2:rot].clone()
                     y[..., :rot // 2] = a * c - b * s_
                     y[..., rot // 2:rot] = a * s_ + b * c
-        qp = torch.zeros(T, nh, D)
-        qp[..., :dk] = q
+        if temperature is not None:
+            steps = torch.div(ctx.positions[:T] + 1, temperature[1], rounding_mode="floor").float()
+            q = q * (1.0 + temperature[0] * torch.log(steps + 1.0))[:, None, None]
+        qp = torch.zeros(T, nh * parts, D)
+        for m in range(parts):
+            qp[:, m::parts, m * dk:(m + 1) * dk] = q[:, m::parts]
+        k = k.reshape(T, nkv, parts * dk)
         valid = (ctx.row_req[:T] >= 0)
         qp[~valid] = 0
-        q_out.copy_(qp.reshape(T, nh * D).to(q_out.dtype))
+        q_out.copy_(qp.reshape(T, nh * parts * D).to(q_out.dtype))
         if not cache.writes:
             return False
         table = ctx.block_tables[cache.group]
@@ -218,7 +244,7 @@ class CpuOps:
             page = int(table[r, pos // P])
             assert page >= 0
             cache.pages[page, :, :, pos % P, :] = 0
-            cache.pages[page, 0, :, pos % P, :dk] = k[t].to(cache.pages.dtype)
+            cache.pages[page, 0, :, pos % P, :k.shape[-1]] = k[t].to(cache.pages.dtype)
             cache.pages[page, 1, :, pos % P, :dv] = v[t].to(cache.pages.dtype)
         return False
 
@@ -307,7 +333,10 @@ class CpuOps:
     def head_norm_gate(self, o, weight, eps, gate, gate0, act, out, heads, vdim, out_col0=0, scale=1.0):
         T = out.shape[0]
         y = o[:T].float().view(T, heads, vdim)
-        w = weight.float().view(heads, vdim)[None] if weight.numel() == heads * vdim else weight.float()[None, None, :]
+        if weight is None:
+            w = 1.0
+        else:
+            w = weight.float().view(heads, vdim)[None] if weight.numel() == heads * vdim else weight.float()[None, None, :]
         y = y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps) * w
         z = gate[:T, gate0:gate0 + heads * vdim].float().view(T, heads, vdim)
         y = y * (z * torch.sigmoid(z) if act == "silu" else torch.sigmoid(z))
@@ -348,6 +377,13 @@ class CpuOps:
                   normalize=True):
         T, E = logits.shape
         z = torch.nan_to_num(logits.float())
+        if score == "softmax_chosen":
+            assert groups == 1
+            z = z + (correction.float()[None, :] if correction is not None else 0.0)
+            top_z, pick = z.topk(top, dim=-1)
+            ids.copy_(pick.to(torch.int32))
+            weights.copy_(torch.softmax(top_z, dim=-1) * scale)
+            return
         s = torch.softmax(z, dim=-1) if score == "softmax" else torch.sigmoid(z)
         choice = s + (correction.float()[None, :] if correction is not None else 0.0)
         if score == "sigmoid" and correction is None and groups == 1:
@@ -598,14 +634,21 @@ class CpuOps:
     def add_rmsnorm_conv(self, branch, weight, eps, residual, conv_weight, state, out, ctx, writes=True):
         return False                                   # the caller runs add_rmsnorm and input_conv
 
-    def decay_memory(self, rows, q0, k0, v0, act, powers, state, out, heads, dim, vdim, ctx, writes=True):
+    def decay_memory(self, rows, q0, k0, v0, act, powers, state, out, heads, dim, vdim, ctx, writes=True,
+                     cos=None, sin=None, rot=0, key_scale=1.0):
+        def turn(x, t):
+            if rot:
+                a, b = x[:, :rot // 2].clone(), x[:, rot // 2:rot].clone()
+                x = torch.cat([a * cos[t] - b * sin[t], b * cos[t] + a * sin[t], x[:, rot:]], dim=1)
+            return x
+
         f = (lambda t: t * torch.sigmoid(t)) if act == "silu" else (lambda t: t)
         a = powers[:, 1][:, None, None]
         for _, mine, slot in self._requests(ctx):
             S = state[slot].clone()
             for t in mine:
-                q = f(rows[t, q0:q0 + heads * dim].float()).view(heads, dim)
-                k = f(rows[t, k0:k0 + heads * dim].float()).view(heads, dim)
+                q = turn(f(rows[t, q0:q0 + heads * dim].float()).view(heads, dim), t)
+                k = turn(f(rows[t, k0:k0 + heads * dim].float()).view(heads, dim), t) * key_scale
                 v = f(rows[t, v0:v0 + heads * vdim].float()).view(heads, vdim)
                 S = a * S + k[:, :, None] * v[:, None, :]
                 out[t] = (S * q[:, :, None]).sum(1).reshape(-1)
