@@ -10,6 +10,7 @@
     python bench.py --compare pimodra
     python bench.py --compare nukelix
     python bench.py --compare lurisun
+    python bench.py --compare fovosun
                     (Bolonex beside Gemma 2, Petanex beside Bolonex, and so on, at equal layer sizes: prefill and decode throughput
                     and, per operation, the time of one step against the time its bytes, or its multiply-adds, take at the
                     measured rates; one JSON line)
@@ -860,6 +861,78 @@ def compare_lurisun(args) -> dict:
                                                                       ("nukelix", nukelix_config(z), nukelix_op_bytes)))
 
 
+# ---- Fovosun beside Petanex, Lurisun and Bolonex at equal layer sizes (--compare fovosun) ------------------------------
+# Eight layers in all four.  Fovosun: differential attention with a convolution and a temperature, differential attention
+# over a window, two retention layers, twice; feed-forwards alternate between dense and a mixture as in Petanex, the closest
+# existing model as a whole; four residual streams.  A head's two maps of dim / 2 have the width of one ordinary head.
+# Lurisun has the like of retention (the same memory with a d x dv state per head), Bolonex the like of the first attention
+# (grouped-query attention behind a convolution over q, k and v).
+FOVOSUN_SIZES = {name: dict(z, window=LURISUN_SIZES[name]["window"], q_rank=LURISUN_SIZES[name]["q_rank"],
+                            kv_rank=LURISUN_SIZES[name]["kv_rank"], streams=4) for name, z in PETANEX_SIZES.items()}
+
+
+def fovosun_config(z: dict) -> dict:
+    d, h = z["dim"], z["d_heads"]
+    att = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": d // 2, "vdim": d, "scale": (d // 2) ** -0.5, "diff": 0.5,
+           "conv": 4, "q_temp": {"coef": 0.1, "every": 1024}}
+    win = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": d // 2, "vdim": d, "scale": (d // 2) ** -0.5, "diff": 0.5,
+           "mask": {"size": z["window"]}, "rot": {"base": 10000.0, "dims": d // 2}}
+    ret = {"heads": h, "dim": z["d_dim"], "vdim": z["d_vdim"], "decay": [1.0 - 2.0 ** -(2.0 + 6.0 * i / h) for i in range(h)],
+           "rot": {"base": 10000.0, "dims": z["d_dim"]}}
+    eff = z["ff"] // (z["top"] + 1) // 64 * 64
+    dense = {"kind": "dense", "ff": z["ff"], "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": eff, "limit": 7.0}, "shared": {"ff": eff, "limit": 7.0},
+           "router": {"experts": z["experts"], "top": z["top"]}}
+    kinds = ["attention", "attention_2", "retention", "retention"]
+    layers = [{"type": kinds[i % 4], "mixer": (att, win, ret, ret)[i % 4], "mlp": dense if i % 2 == 0 else moe}
+              for i in range(COMPARE_LAYERS)]
+    return {"architecture": "Fovosun", "width": z["width"], "vocab": COMPARE_VOCAB, "streams": z["streams"],
+            "embedding": {"scale": 1.0}, "norm": {"eps": 1e-5}, "layers": layers}
+
+
+def fovosun_op_bytes(z: dict, T: int, n_reqs: int, keys: int) -> dict:
+    """Bytes (and, for the products, floating-point operations) each operation of one Fovosun step must move, summed over
+    the layers that use it; a prompt's attention also has the multiply-adds of the keys its rows see, those of the zero
+    halves of its query rows not counted."""
+    W, H, G, dv, L, n = z["width"], z["heads"], z["kv_heads"], z["dim"], COMPARE_LAYERS, z["streams"]
+    d = dv // 2
+    n_full, n_win, n_ret, n_moe = L // 4, L // 4, L // 2, L // 2
+    mh, md, mv = z["d_heads"], z["d_dim"], z["d_vdim"]
+    single = T == n_reqs
+    cq = 2 * (H + G) * d + G * dv
+    seen = min(keys, z["window"])
+    pairs = n_reqs * keys if single else T * (T + 1) // 2
+    pairs_w = n_reqs * seen if single else sum(min(i + 1, z["window"]) for i in range(T))
+    eff = z["ff"] // (z["top"] + 1) // 64 * 64
+    P = T * z["top"]
+    used = min(z["experts"], P)
+    return {
+        "embed": T * W * (2 + 4 * n),
+        "streams_step": 2 * L * T * W * (8 * n + 6),
+        "streams_norm": T * W * (4 * n + 2) + n_reqs * W * (4 * n + 2),
+        "qkv_prepare": (n_full + n_win) * T * 6 * cq + n_win * T * 4 * d,
+        "short_conv_commit": n_full * n_reqs * 3 * cq * 8,
+        "paged_attention": ((n_full * keys + n_win * seen) * n_reqs * G * (2 * d + dv) * 2 + (n_full + n_win) * T * H * (2 * d + 2 * dv) * 2,
+                            4 * H * (d + dv) * (n_full * pairs + n_win * pairs_w)),
+        "diff_combine": (n_full + n_win) * T * H * dv * 6,
+        "decay_rotate": n_ret * T * (mh * (2 * md + mv) * 6 + 4 * md),
+        "decay_memory": n_ret * (T * mh * (2 * md + mv) * (4 if single else 2) + T * mh * mv * 4 + 2 * n_reqs * mh * md * mv * 4),
+        "head_norm_gate": n_ret * T * mh * mv * 10,
+        "linear_gated": ((L - n_moe) * (2 * z["ff"] * W * 2 + T * (2 * W + 2 * z["ff"])) + n_moe * (2 * eff * W * 2 + T * (2 * W + 2 * eff)),
+                         4 * T * W * ((L - n_moe) * z["ff"] + n_moe * eff)),
+        "moe_route": n_moe * T * (z["experts"] * 4 + z["top"] * 8),
+        "moe_plan": n_moe * P * 12,
+        "moe_linear": (n_moe * (used * 3 * eff * W * 2 + P * (2 * W + 4 * eff + 4 * W)), n_moe * 6 * P * eff * W),
+        "moe_combine": n_moe * T * W * (4 * z["top"] + 8),
+    }
+
+
+def compare_fovosun(args) -> dict:
+    return compare_models(args, "fovosun", FOVOSUN_SIZES, lambda z: (
+        ("fovosun", fovosun_config(z), fovosun_op_bytes), ("petanex", petanex_config(z), petanex_op_bytes),
+        ("lurisun", lurisun_config(z), lurisun_op_bytes), ("bolonex", bolonex_config(z), bolonex_op_bytes)))
+
+
 def micro_attention() -> int:
     """Decode attention alone: eight launches over distinct pages replayed from a CUDA graph, per batch size; one JSON
     line each with microseconds per launch and bytes of keys and values over that time."""
@@ -1314,15 +1387,16 @@ def main() -> int:
     ap.add_argument("--only-headline", action="store_true", help="skip the other batch sizes, the mixed steps, 32-bit and the other model sizes")
     ap.add_argument("--micro", choices=["attention", "prompt-attention", "gemm", "products", "qkv-rope", "reference", "memory"],
                     help="time kernels alone instead of the model step")
-    ap.add_argument("--compare", choices=["bolonex", "petanex", "pimodra", "nukelix", "lurisun"],
-                    help="another workload: Bolonex beside Gemma 2, Petanex beside Bolonex, Pimodra beside Gemma 2, Nukelix beside Petanex, or Lurisun beside Nukelix, at equal "
+    ap.add_argument("--compare", choices=["bolonex", "petanex", "pimodra", "nukelix", "lurisun", "fovosun"],
+                    help="another workload: Bolonex beside Gemma 2, Petanex beside Bolonex, Pimodra beside Gemma 2, Nukelix beside Petanex, Lurisun beside Nukelix, or "
+                         "Fovosun beside Petanex, Lurisun and Bolonex, at equal "
                          "layer sizes (prefill, decode, per-operation rooflines)")
     args = ap.parse_args()
     if args.compare:
         args.warmup = max(args.warmup, 3)
         args.reps = max(args.reps, 1)
         print(json.dumps({"bolonex": compare_bolonex, "petanex": compare_petanex, "pimodra": compare_pimodra,
-                          "nukelix": compare_nukelix, "lurisun": compare_lurisun}[args.compare](args)))
+                          "nukelix": compare_nukelix, "lurisun": compare_lurisun, "fovosun": compare_fovosun}[args.compare](args)))
         return 0
     if args.micro:
         return {"attention": micro_attention, "prompt-attention": micro_prompt_attention, "gemm": micro_gemm,

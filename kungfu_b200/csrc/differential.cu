@@ -14,7 +14,15 @@ template <int V> __device__ __forceinline__ void df_load(const float* p, float* 
   else v[0] = *p;
 }
 template <int V> __device__ __forceinline__ void df_load(const __nv_bfloat16* p, float* v) {
-  if constexpr (V == 4) {
+  if constexpr (V == 8) {
+    const uint4 r = *reinterpret_cast<const uint4*>(p);
+    const uint32_t u[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u[k]));
+      v[2 * k] = f.x, v[2 * k + 1] = f.y;
+    }
+  } else if constexpr (V == 4) {
     const uint2 r = *reinterpret_cast<const uint2*>(p);
     const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x));
     const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
@@ -28,7 +36,15 @@ template <int V> __device__ __forceinline__ void df_store(float* p, const float*
   else *p = v[0];
 }
 template <int V> __device__ __forceinline__ void df_store(__nv_bfloat16* p, const float* v) {
-  if constexpr (V == 4) {
+  if constexpr (V == 8) {
+    uint32_t u[4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const __nv_bfloat162 h = __floats2bfloat162_rn(v[2 * k], v[2 * k + 1]);
+      u[k] = *reinterpret_cast<const uint32_t*>(&h);
+    }
+    *reinterpret_cast<uint4*>(p) = make_uint4(u[0], u[1], u[2], u[3]);
+  } else if constexpr (V == 4) {
     const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
     *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
   } else {
@@ -100,6 +116,13 @@ int diff_go(const void* o, float lambda, float factor, float eps, const float* g
 #define KF_GO(V, L)                                                                                                        \
   kf_launch(diff_combine_kernel<T, V, L>, dim3((unsigned)kf_ceil_div((long)rows * nh, DF_THREADS / L)), dim3(DF_THREADS), 0, stream, \
             (const T*)o, lambda, factor, eps, g, ld, gcol0, nh, dv, D, (T*)out, row_req, rows)
+  if constexpr (sizeof(T) == 2) {
+    if (by4 && dv % 8 == 0 && D % 8 == 0) {                // 16 bytes per lane and load
+      if (dv <= 64) KF_GO(8, 8); else if (dv <= 128) KF_GO(8, 16); else KF_GO(8, 32);
+      KF_CHECK_LAUNCH();
+      return KF_OK;
+    }
+  }
   if (!by4) KF_GO(1, 32);
   else if (dv <= 32) KF_GO(4, 8);
   else if (dv <= 64) KF_GO(4, 16);

@@ -315,6 +315,24 @@ qkv_prepare_halves_kernel(KfConvIn cv, const TW* __restrict__ conv_w, const TW* 
   const float* sn = sin_t + (size_t)t * half;
   const float temp = qp_temperature(temp_coef, temp_every, pos);
   float* xs = hs[warp];
+  // of this lane's elements 4 lane + 128 r .. + 3 of any head of q or k: the part, the partner's distance (0: not turned)
+  // and the angles, the same for every head of the row
+  int part[NR], pair[NR];
+  float4 cc[NR], sv[NR];
+#pragma unroll
+  for (int r = 0; r < NR; ++r) {
+    const int i = 4 * lane + 128 * r;
+    const bool in_head = i < parts * dk;
+    part[r] = in_head ? i / dk : 0;
+    const int e = i - part[r] * dk;
+    pair[r] = (in_head && e < rot) ? (e < half ? half : -half) : 0;
+    if (pair[r] != 0) {
+      const int at = pair[r] > 0 ? e : e - half;
+      cc[r] = *reinterpret_cast<const float4*>(c + at);
+      sv[r] = *reinterpret_cast<const float4*>(sn + at);
+      if (pair[r] > 0) sv[r] = make_float4(-sv[r].x, -sv[r].y, -sv[r].z, -sv[r].w);
+    }
+  }
   for (int hslot = blockIdx.y * QP_WARPS + warp; hslot < slots; hslot += stride) {
     const int kind = hslot < nh ? 0 : (hslot < nh + nkv ? 1 : 2);
     const int head = kind == 0 ? hslot : (kind == 1 ? hslot - nh : hslot - nh - nkv);
@@ -356,20 +374,16 @@ qkv_prepare_halves_kernel(KfConvIn cv, const TW* __restrict__ conv_w, const TW* 
       const int i = 4 * lane + 128 * r;
       if (i >= D) continue;
       float4 v = x[r];                                      // zero beyond d
-      const int part = (kind == 2 || i >= d) ? 0 : i / dk, e = i - part * dk;
-      if (turned && i < d && e < rot) {
-        const bool low = e < half;
-        const float4 y = *reinterpret_cast<const float4*>(xs + (low ? i + half : i - half));
-        const float4 cc = *reinterpret_cast<const float4*>(c + (low ? e : e - half));
-        float4 sv = *reinterpret_cast<const float4*>(sn + (low ? e : e - half));
-        if (low) sv = make_float4(-sv.x, -sv.y, -sv.z, -sv.w);
-        v = make_float4(fmaf(v.x, cc.x, y.x * sv.x), fmaf(v.y, cc.y, y.y * sv.y), fmaf(v.z, cc.z, y.z * sv.z), fmaf(v.w, cc.w, y.w * sv.w));
+      if (turned && pair[r] != 0) {
+        const float4 y = *reinterpret_cast<const float4*>(xs + i + pair[r]);
+        v = make_float4(fmaf(v.x, cc[r].x, y.x * sv[r].x), fmaf(v.y, cc[r].y, y.y * sv[r].y), fmaf(v.z, cc[r].z, y.z * sv[r].z),
+                        fmaf(v.w, cc[r].w, y.w * sv[r].w));
       }
       if (kind == 0) {
         v.x *= f; v.y *= f; v.z *= f; v.w *= f;
         const size_t at = ((size_t)t * nh + head) * parts * D + i;
         for (int m = 0; m < parts; ++m)
-          kf_store_vec4(q_out, at + (size_t)m * D, m == part ? v : make_float4(0.f, 0.f, 0.f, 0.f));
+          kf_store_vec4(q_out, at + (size_t)m * D, m == part[r] ? v : make_float4(0.f, 0.f, 0.f, 0.f));
       } else {
         kf_store_vec4(pages, ((((size_t)page * 2 + (kind - 1)) * nkv + head) * page_size + (pos % page_size)) * D + i, v);
       }

@@ -184,6 +184,11 @@ def build(cfg: FovosunConfig, w: WeightStore) -> DecoderModel:
         if l.mlp is not None:
             ffn = _feed_forward(cfg, w, l.mlp, p + "mlp.")
             norm2, mix2 = sublayer(p, 2)
+        else:                                       # a file may still hold the numbers of a sublayer that does not run
+            unused = [s.name for s in _streams_specs(cfg, p, 2) if w.has(s.name)]
+            for name in unused:
+                w.take(name, w.shape_of(name))
+            w.release(*unused)
         if w.faulty:
             w.finish()
         blocks.append(StreamsBlock(norm1, mixer, mix1, norm2, ffn, mix2))

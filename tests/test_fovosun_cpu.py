@@ -102,6 +102,12 @@ def test_weights_bind_by_name_and_faults_are_listed_together():
     c = api.load_config(json.loads(json.dumps(fo.FO_C)))                # one tap: no tail
     one = arch.build(c, WeightStore.from_tensors(fo.draw_tensors(fo.FO_C, 1), device="cpu", compute_dtype=torch.float32))
     assert one.state_needs()[0].n_kv_heads == 1 and one.layers[0].mixer.conv.taps == 1
+    # the numbers of a second sublayer that layer 1 does not have may stand in the file; anything else may not
+    arch.build(cfg, WeightStore.from_tensors(dict(t, **{"l1.hc2.in": torch.zeros(2), "l1.norm2": torch.zeros(64)}), device="cpu",
+                                             compute_dtype=torch.float32))
+    with pytest.raises(WeightError) as e:
+        arch.build(cfg, WeightStore.from_tensors(dict(t, **{"l1.mlp.up": torch.zeros(4, 64)}), device="cpu", compute_dtype=torch.float32))
+    assert e.value.unexpected == ["l1.mlp.up"]
     bad = dict(t)
     del bad["l1.mix.g"]
     with pytest.raises(WeightError) as e:

@@ -130,8 +130,10 @@ MAP_SHAPES = [  # H, G, d, dv, taps, rot, temperature, biased, page
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("lengths,sizes", [([37, 25], [(1, 2), (5, 1), (1, 1), (1, 1), (2, 9), (1, 1), (11, 3)]),
+                                           ([690, 205], [(1, 2), (550, 7), (1, 1), (3, 190), (9, 2)])])
 @pytest.mark.parametrize("H,G,d,dv,taps,rot,temp,biased,P", MAP_SHAPES)
-def test_queries_and_keys_of_two_maps_in_portions(dtype, H, G, d, dv, taps, rot, temp, biased, P):
+def test_queries_and_keys_of_two_maps_in_portions(dtype, H, G, d, dv, taps, rot, temp, biased, P, lengths, sizes):
     """Two requests fed in portions of changing size (single rows also move the convolution's tail in the same kernel where
     they can): every query row is its map's query in its own half and zero elsewhere, the stored key is both maps side by
     side, the value is filed once, tails are zero, and a padding row leaves nothing."""
@@ -142,7 +144,7 @@ def test_queries_and_keys_of_two_maps_in_portions(dtype, H, G, d, dv, taps, rot,
     g = torch.Generator().manual_seed(H * d + dv + taps)
     C, D = 2 * (H + G) * d + G * dv, latent_head_size(max(2 * d, dv))
     ld = C + (-C) % 4
-    lengths, slots = [37, 25], [2, 0]
+    slots = [2, 0]
     raw = [torch.randn(n, ld, generator=g) for n in lengths]
     bias = (0.4 * torch.randn(C, generator=g)).to(tdt) if biased else None
     conv = (0.6 * torch.randn(C, taps, generator=g)).to(tdt) if taps else None
@@ -159,13 +161,12 @@ def test_queries_and_keys_of_two_maps_in_portions(dtype, H, G, d, dv, taps, rot,
         for m in (0, 1):
             wide[:, :, m, m * d:(m + 1) * d] = q.view(n, H, 2, d)[:, :, m]
         want.append((wide.view(n, 2 * H, D), k.reshape(n, G, 2 * d), u[:, 2 * (H + G) * d:].reshape(n, G, dv)))
-    table = torch.arange(2 * (40 // P + 2), dtype=torch.int32).view(2, -1).flip(1).contiguous()
+    table = torch.arange(2 * (max(lengths) // P + 2), dtype=torch.int32).view(2, -1).flip(1).contiguous()
     pages = torch.full((table.numel(), 2, G, P, D), 7.0, dtype=tdt, device=DEV)
     cache = types.SimpleNamespace(pages=pages, page_size=P, group=0, writes=True)
     state = torch.zeros(3, max(taps - 1, 1), C, device=DEV)
     half = 50.0 ** (-2.0 * torch.arange(rot // 2, dtype=torch.float64) / max(rot, 1))
     done, step, inline_seen = [0, 0], 0, False
-    sizes = [(1, 2), (5, 1), (1, 1), (1, 1), (2, 9), (1, 1), (11, 3)]
     while min(a - b for a, b in zip(done, lengths)) < 0:
         rows = [min(s, n - a) for s, n, a in zip(sizes[step % len(sizes)], lengths, done)]
         step += 1
@@ -192,12 +193,12 @@ def test_queries_and_keys_of_two_maps_in_portions(dtype, H, G, d, dv, taps, rot,
             at += n
             done[r] += n
         assert float(q[at:].abs().max()) == 0.0
+    pages = pages.cpu()
     for r, n in enumerate(lengths):
-        for j in range(n):
-            page = int(table[r, j // P])
-            kk, vv = pages[page, 0, :, j % P], pages[page, 1, :, j % P]
-            assert _rel(kk[:, :2 * d], want[r][1][j]) < tol and _rel(vv[:, :dv], want[r][2][j]) < tol, (r, j)
-            assert float(kk[:, 2 * d:].abs().sum()) == 0.0 and float(vv[:, dv:].abs().sum()) == 0.0
+        at = torch.arange(n)
+        kk, vv = (pages[table[r, at // P].long(), i, :, at % P] for i in (0, 1))
+        assert _rel(kk[..., :2 * d], want[r][1]) < tol and _rel(vv[..., :dv], want[r][2]) < tol, r
+        assert float(kk[..., 2 * d:].abs().sum()) == 0.0 and float(vv[..., dv:].abs().sum()) == 0.0
     assert inline_seen == (taps > 1 and d % 4 == 0 and dv % 4 == 0 and rot % 8 == 0)
 
 
