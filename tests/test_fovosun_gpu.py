@@ -84,7 +84,7 @@ def _step_ctx(rows_of_reqs, slots, pad_rows=0, starts_at=None):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("n,W,T", [(1, 64, 3), (2, 30, 5), (3, 320, 200), (4, 2048, 40), (5, 101, 2), (6, 96, 7), (7, 64, 4), (8, 512, 9),
+@pytest.mark.parametrize("n,W,T", [(1, 64, 3), (2, 30, 5), (3, 328, 200), (4, 2048, 40), (5, 101, 2), (6, 96, 7), (7, 64, 4), (8, 512, 9),
                                    (16, 36, 5), (11, 7, 3), (3, 4100, 2)])
 def test_streams_update_and_reading(dtype, n, W, T):
     """The update alone, the update with the next sublayer's reading, and the reading alone of some rows."""
@@ -123,7 +123,7 @@ def test_embedding_starts_every_stream(dtype):
 
 
 MAP_SHAPES = [  # H, G, d, dv, taps, rot, temperature, biased, page
-    (4, 2, 32, 64, 3, 0, (0.5, 16), False, 64), (4, 1, 32, 64, 0, 32, None, True, 64), (2, 2, 8, 20, 4, 8, (0.3, 1), True, 8),
+    (6, 2, 32, 64, 3, 0, (0.6, 16), False, 64), (5, 1, 32, 48, 0, 32, None, True, 64), (2, 2, 8, 20, 4, 8, (0.3, 1), True, 8),
     (6, 3, 16, 16, 2, 8, None, False, 16), (3, 1, 9, 7, 3, 4, (1.1, 3), True, 4), (2, 1, 64, 128, 4, 64, (0.4, 100), False, 64),
     (1, 1, 104, 40, 1, 16, None, False, 64), (2, 2, 136, 100, 3, 136, (0.2, 7), True, 64), (2, 1, 6, 30, 8, 2, None, False, 16),
     (4, 4, 20, 12, 5, 16, (0.7, 9), True, 32), (2, 1, 24, 300, 2, 12, None, False, 16)]
@@ -237,7 +237,7 @@ def test_preparation_of_one_map_with_norms(dtype, interleaved, rot, norm):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("H,G,d,dv,P,window", [(4, 2, 32, 64, 64, None), (4, 1, 32, 64, 64, 70), (8, 1, 16, 24, 16, 33), (9, 1, 64, 128, 64, 40),
+@pytest.mark.parametrize("H,G,d,dv,P,window", [(6, 2, 32, 64, 64, None), (5, 1, 32, 48, 64, 70), (8, 1, 16, 24, 16, 33), (9, 1, 64, 128, 64, 40),
                                                (2, 2, 64, 40, 64, 1), (3, 3, 10, 30, 8, None), (2, 1, 128, 256, 64, 100), (2, 1, 140, 60, 64, 50)])
 @pytest.mark.parametrize("fast", [True, False])
 def test_both_maps_on_the_attention_kernels_and_their_difference(dtype, H, G, d, dv, P, window, fast, monkeypatch):
@@ -428,7 +428,7 @@ def _check(got, ref, tol, noisy=None):
 ONE_LAYER = {
     "plain_maps": fo.config(64, 200, [fo.layer("attention_2", fo.attention(4, 2, 12, 16, 0.4))]),
     "window": fo.config(64, 200, [fo.layer("attention_2", fo.attention(4, 4, 32, 64, 0.3, window=37, rot=(100.0, 16)))], streams=1),
-    "conv_temperature": fo.config(64, 200, [fo.layer("attention", fo.attention(4, 2, 32, 64, 0.2, conv=4, temp=(0.6, 9)))], streams=4),
+    "conv_temperature": fo.config(64, 200, [fo.layer("attention", fo.attention(6, 2, 32, 64, 0.2, conv=4, temp=(0.6, 9)))], streams=4),
     "many_heads": fo.config(64, 200, [fo.layer("attention_2", fo.attention(10, 1, 8, 16, 0.5, window=50, rot=(10.0, 8)))]),
     "taps": fo.config(64, 200, [fo.layer("attention", fo.attention(1, 1, 9, 8, 0.5, conv=8, temp=(0.2, 1)))], streams=2),
     "wide_maps": fo.config(128, 200, [fo.layer("attention", fo.attention(2, 1, 128, 200, 0.1, conv=2, temp=(0.3, 64)))]),
